@@ -82,7 +82,7 @@ int pg_gemm_bf16(const void* x, long long ldx, const void* w, long long ldw, voi
  *  - out_row_map (token-major kernels, PG_EPI_F32 without resid): token t is written to output row out_row_map[t] -- the
  *    multimodal projector (modeling_paligemma.py:57-65) scattering its rows, times `scale`, straight to the `<image>` positions of
  *    the merged embedding sequence (masked_scatter of _merge_input_ids_with_image_features, :201-251); map from pg_merge_scan.
- *  - PG_EPI_GEGLU takes the kind of gated unit from act_gelu: 0 / 1 gelu_tanh(g) * u, 3 silu(g) * u, 4 the clamped form
+ *  - PG_EPI_GEGLU takes the kind of gated unit from act_gelu: 0 / 1 gelu_tanh(g) * u, 3 silu(g) * u, 5 relu(g) * u, 4 the clamped form
  *    g' = min(g, c), u' = clamp(u, -c, c), g' * sigmoid(glu_alpha * g') * (u' + 1) with c = `scale` (glu_alpha 0 reads as 1).  In this
  *    mode `bias` (fp32 [features]) is in the packed row order of the weight ([64 gate | 64 up] per 128 rows) and is added before
  *    the gated unit.
@@ -372,7 +372,11 @@ int pg_attn_prepare(const void* qkv, long long ld, const int* pos, const int* ro
  *                   keep their true positions);
  *   sink            [H] fp32: exp(sink[h]) joins the softmax denominator once, with no key, no value and no scale;
  *   dist_a, dist_b  [H] fp32 each: the score loses dist_a[h] * log(1 + dist_b[h] * (i - j));
- *   head_scale      [H] fp32: the scaled dot product is multiplied by head_scale[h] (before the distance term is taken off). */
+ *   head_scale      [H] fp32: the scaled dot product is multiplied by head_scale[h] (before the distance term is taken off);
+ *   logistic        no softmax: the weight of a visible key is 1 / (1 + exp(-(score + head_bias[h]))) and the weights are not normalised
+ *                   over the keys (head_bias [H] fp32 or NULL; no sink); dim, vdim as for the softmax form;
+ *   out_scale       != 0: the output is multiplied by it;
+ *   out_ld          != 0: elements between consecutive rows of `out` (0: H * vdim). */
 typedef struct PgAttnScore {
   int window;
   int keep_first;
@@ -380,6 +384,10 @@ typedef struct PgAttnScore {
   const float* dist_a;
   const float* dist_b;
   const float* head_scale;
+  int logistic;
+  const float* head_bias;
+  float out_scale;
+  long long out_ld;
 } PgAttnScore;
 
 /* Causal attention of every entry's new rows over its cached keys / values (query head h reads k/v head h / (H / G)):
@@ -435,6 +443,79 @@ int pg_linear_attn_scan(const void* qkv, long long ld, float* state, const float
 int pg_linear_attn_chunked(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* entry_row0,
                            const int* entry_n, const int* entry_ctx, const int* entry_slot, int entries, int H, int dim, int vdim,
                            int act_f32, void* stream);
+
+/* ---- recurrent mixers: a matrix state per head and sequence in fp32 ------------------------------------------------------------
+ * Entry e continues slot entry_slot[e] (from zero when entry_ctx[e] == 0) and leaves its new state there.
+ *
+ * pg_short_conv: per channel c, y[t] = silu(sum_j w[j * C + c] * x[t - taps + 1 + j] + bias[c]), zeros before the sequence's start; the
+ * last taps - 1 inputs live in state fp32 [slots, taps - 1, C] (taps <= 8; taps == 1: no state).  Channels come in up to three sections:
+ * section s holds `groups` groups of `size` channels (`total` channels; the last group may be short), its inputs start at column
+ * xcol of x, its weights, state and outputs at channel ccol.  unit != 0: inv[t * ldi + group] = scale / sqrt(sum over the group of y^2 +
+ * 1e-6), groups numbered over the unit sections in order. */
+typedef struct PgConvSections {
+  int count;
+  int groups[3], size[3], total[3], xcol[3], ccol[3], unit[3];
+  float scale[3];
+} PgConvSections;
+int pg_short_conv(const void* x, long long ldx, const float* w, const float* bias, float* state, void* out, long long ldo, float* inv, int ldi,
+                  const PgConvSections* sections, int taps, int C, const int* entry_row0, const int* entry_n, const int* entry_ctx,
+                  const int* entry_slot, int entries, int max_n, int act_f32, void* stream);
+
+/* Delta rule, one decay per head and key channel.  Row t, head h (hk = h / (H / G)): q = q[t * ldq + hk * dim ..] * inv[t * ldi + hk], k likewise
+ * with inv[t * ldi + G + hk], v = v[t * ldv + h * vdim ..], b = sigmoid(beta[t * ldb + h]), g[d] = exp(-exp(A_log[h]) *
+ * softplus(decay[t * lda + h * dim + d] + dt_bias[h * dim + d])) (decay fp32);
+ *   S[d, :] <- g[d] S[d, :];  u = b (v - S^T k);  S <- S + k u^T;  out[t, h * vdim ..] = S^T q   (fp32, pitch H * vdim).
+ * state fp32 [slots, H, dim, vdim].  q, k, v, beta: activation type. */
+typedef struct PgDeltaArgs {
+  const void *q, *k, *v, *beta;
+  long long ldq, ldk, ldv, ldb;
+  const float* inv;
+  int ldi;
+  const float* decay;
+  long long lda;
+  const float *A_log, *dt_bias;
+  float* state;
+  float* out;
+  const int *entry_row0, *entry_n, *entry_ctx, *entry_slot;
+  int entries, H, G, dim, vdim;
+} PgDeltaArgs;
+
+/* Recurrences with one scalar decay per head and token: S <- keep * S + put * k v^T, read out with q (k, q of group h / (H / G)).
+ * kind 0, state space: dt = softplus(gate1[t * ldg + h] + p1[h]), keep = exp(-exp(p2[h]) dt), put = dt, out = S^T q + p3[h] v.
+ * kind 1, matrix memory: i = cap tanh((gate1 + p1[h]) / cap), f = log sigmoid(cap tanh((gate2 + p2[h]) / cap)); running maximum
+ *   m' = max(f + m, i) from m = 0; keep = exp(f + m - m'), put = exp(i - m'); n <- keep n + put k;
+ *   out = S^T q / (max(|n . q|, exp(-m')) + 1e-6), q multiplied by qscale.
+ * state fp32 [slots, H, dim, vdim]; norm_state (kind 1) fp32 [slots, ceil(vdim / pg_recurrence_block(vdim)), H, dim + 1]: n and m, one
+ * copy per block of value columns. */
+typedef struct PgGatedArgs {
+  const void *q, *k, *v;
+  long long ldq, ldk, ldv;
+  float qscale;
+  const void *gate1, *gate2;
+  long long ldg;
+  const float *p1, *p2, *p3;
+  float cap;
+  float *state, *norm_state;
+  float* out;
+  const int *entry_row0, *entry_n, *entry_ctx, *entry_slot;
+  int entries, H, G, dim, vdim;
+} PgGatedArgs;
+int pg_recurrence_block(int vdim);
+/* Token by token; entries with fewer than n_min or more than n_max new tokens are left alone (another form advances them). */
+int pg_delta_scan(const PgDeltaArgs* args, int n_min, int n_max, int act_f32, void* stream);
+int pg_gated_scan(const PgGatedArgs* args, int kind, int n_min, int n_max, int act_f32, void* stream);
+
+/* out[t, :] = scale * G(o[t, :]) with G a norm in `groups` equal consecutive parts (each divided by its own root mean square) times w and a
+ * gate: gate_mode 1 -- norm(o) * w * sigmoid(gate); 2 -- norm(o * silu(gate)) * w; 0 -- no gate.  w_n == D: a weight per column;
+ * w_n == D / groups: shared by the groups.  o fp32 [rows, D]; gate, out: activation type (pitches ldg, ldo). */
+int pg_group_norm_gate(const float* o, const float* w, int w_n, const void* gate, long long ldg, int gate_mode, void* out, long long ldo, int rows,
+                       int D, int groups, float eps, float scale, int act_f32, void* stream);
+
+/* A gated sub-layer result joins the residual behind a layer norm, and the next sub-layer's input norm follows from the same row:
+ *   z = y[t, :] * sigmoid(gate[t, :] + gate_b);  x[t, :] += LN(z; w1, b1);  out[t, :] = LN(x[t, :]; w2, b2)   (out NULL: no second norm)
+ * y fp32 (pitch ldy), gate activation type (pitch ldg; NULL: no gate), x fp32 [rows, D] in place, out activation type [rows, D]. */
+int pg_gated_layernorm_add(const float* y, long long ldy, const void* gate, long long ldg, const float* gate_b, const float* w1, const float* b1, float* x,
+                           const float* w2, const float* b2, void* out, int rows, int D, float eps, int act_f32, void* stream);
 
 /* ---- multi-stream residual ("hyper-connections"): xs fp32 [rows, S, D], S <= 16 ------------------------------------------------
  * pg_embed_streams: xs[t, s, :] = table[tokens[t], 0:D] * scale for every stream s.

@@ -13,7 +13,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("PG_LIB_PATH") or os.path.join(_HERE, "libpaligemma_b200.so")  # PG_LIB_PATH: A/B builds (profiling)
 
 EPI_BF16, EPI_F32, EPI_ATOMIC_F32, EPI_GEGLU = 0, 1, 2, 3
-ABI_VERSION = 4  # pg_abi_version() of the library these signatures describe
+ABI_VERSION = 5  # pg_abi_version() of the library these signatures describe
 
 _ERRORS = {-1: "PG_ERR_ARG", -2: "PG_ERR_CUDA", -3: "PG_ERR_DRIVER", -4: "PG_ERR_TMAP", -5: "PG_ERR_ARCH"}
 
@@ -98,6 +98,12 @@ SIGNATURES = {
     "pg_polynorm": [p, i64, p, p, i64, i32, i32, f32, i32, p],
     "pg_sigmoid_gate_mul": [p, i64, p, i64, i32, i32, i32, p],
     "pg_layernorm_shift": [p, p, p, p, p, p, p, p, p, p, p, p, p, p, i32, i32, f32, i32, p],
+    "pg_short_conv": [p, i64, p, p, p, p, i64, p, i32, p, i32, i32, p, p, p, p, i32, i32, i32, p],
+    "pg_recurrence_block": [i32],
+    "pg_delta_scan": [p, i32, i32, i32, p],
+    "pg_gated_scan": [p, i32, i32, i32, i32, p],
+    "pg_group_norm_gate": [p, p, i32, p, i64, i32, p, i64, i32, i32, i32, f32, f32, i32, p],
+    "pg_gated_layernorm_add": [p, i64, p, i64, p, p, p, p, p, p, p, i32, i32, f32, i32, p],
     "pg_glu": [p, i64, p, i64, i32, i32, i32, f32, f32, i32, p],
 }
 _RESTYPE = {"pg_launch_count": i64}
@@ -106,7 +112,28 @@ _RESTYPE = {"pg_launch_count": i64}
 
 class AttnScore(C.Structure):
     """Mirror of PgAttnScore (include/paligemma_b200.h): the optional parts of an attention's score and mask."""
-    _fields_ = [("window", i32), ("keep_first", i32), ("sink", p), ("dist_a", p), ("dist_b", p), ("head_scale", p)]
+    _fields_ = [("window", i32), ("keep_first", i32), ("sink", p), ("dist_a", p), ("dist_b", p), ("head_scale", p), ("logistic", i32),
+                ("head_bias", p), ("out_scale", f32), ("out_ld", i64)]
+
+
+class ConvSections(C.Structure):
+    """Mirror of PgConvSections (include/paligemma_b200.h)."""
+    _fields_ = [("count", i32)] + [(n, i32 * 3) for n in ("groups", "size", "total", "xcol", "ccol", "unit")] + [("scale", f32 * 3)]
+
+
+class DeltaArgs(C.Structure):
+    """Mirror of PgDeltaArgs."""
+    _fields_ = ([(n, p) for n in ("q", "k", "v", "beta")] + [(n, i64) for n in ("ldq", "ldk", "ldv", "ldb")] + [("inv", p), ("ldi", i32), ("decay", p), ("lda", i64)]
+                + [(n, p) for n in ("A_log", "dt_bias", "state", "out", "entry_row0", "entry_n", "entry_ctx", "entry_slot")]
+                + [(n, i32) for n in ("entries", "H", "G", "dim", "vdim")])
+
+
+class GatedArgs(C.Structure):
+    """Mirror of PgGatedArgs."""
+    _fields_ = ([(n, p) for n in ("q", "k", "v")] + [(n, i64) for n in ("ldq", "ldk", "ldv")] + [("qscale", f32), ("gate1", p), ("gate2", p), ("ldg", i64)]
+                + [(n, p) for n in ("p1", "p2", "p3")] + [("cap", f32)]
+                + [(n, p) for n in ("state", "norm_state", "out", "entry_row0", "entry_n", "entry_ctx", "entry_slot")]
+                + [(n, i32) for n in ("entries", "H", "G", "dim", "vdim")])
 
 
 class GemmFusion(C.Structure):
@@ -171,7 +198,7 @@ def require_device():
 # ------------------------------------------------------------------------------------------------------------------
 # thin typed wrappers (argument checking that needs tensor metadata lives here; kernels check the rest)
 # ------------------------------------------------------------------------------------------------------------------
-GLU_GELU, GLU_SILU, GLU_CLAMPED = 1, 3, 4  # gated units of the EPI_GEGLU epilogue (passed as act_gelu)
+GLU_GELU, GLU_SILU, GLU_CLAMPED, GLU_RELU = 1, 3, 4, 5  # gated units of the EPI_GEGLU epilogue (passed as act_gelu)
 
 
 def gemm(x, w, out, *, mode, bias=None, resid=None, act_gelu=0, scale=1.0, swap=-1, split_k=1, features=None, resid_row_mod=0,

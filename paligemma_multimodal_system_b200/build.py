@@ -45,13 +45,28 @@ def build(force: bool = False, verbose: bool = False) -> str:
     nvcc = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
     extra = ["-Xptxas", "-v"] if verbose else []
 
+    headers = hashlib.sha256()
+    for root in (CSRC, INCLUDE):
+        for f in sorted(os.listdir(root)):
+            if f.endswith((".cuh", ".h")):
+                headers.update(open(os.path.join(root, f), "rb").read())
+
     def compile_one(src):
+        """One object per source, recompiled when the source, any header or the flags changed."""
         obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
+        h = headers.copy()
+        h.update(open(src, "rb").read())
+        h.update(" ".join(NVCC_FLAGS).encode())
+        mark = obj + ".stamp"
+        if not force and not verbose and os.path.exists(obj) and os.path.exists(mark) and open(mark).read() == h.hexdigest():
+            return obj
         r = subprocess.run([nvcc, *NVCC_FLAGS, *extra, "-c", src, "-o", obj], capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"nvcc failed for {src}:\n{r.stdout}\n{r.stderr}")
         if verbose:
             sys.stderr.write(r.stderr)
+        with open(mark, "w") as f:
+            f.write(h.hexdigest())
         return obj
 
     with ThreadPoolExecutor(max_workers=8) as ex:

@@ -135,7 +135,7 @@ PG_DEVINL float epilogue_act(float x, int act) {
   return gelu_tanh_fast(x);
 }
 
-// gated unit of the GEGLU epilogue (GemmArgs::act_gelu in that mode): 0 / 1 gelu_tanh(g) * u; 3 silu(g) * u;
+// gated unit of the GEGLU epilogue (GemmArgs::act_gelu in that mode): 0 / 1 gelu_tanh(g) * u; 3 silu(g) * u; 5 relu(g) * u;
 // 4 clamped: g' = min(g, c), u' = clamp(u, -c, c), g' * sigmoid(alpha * g') * (u' + 1) with c = GemmArgs::scale
 PG_DEVINL float glu_act(float g, float u, int kind, float limit, float alpha) {
   if (kind == 3) return g / (1.0f + __expf(-g)) * u;
@@ -144,6 +144,7 @@ PG_DEVINL float glu_act(float g, float u, int kind, float limit, float alpha) {
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.0f + __expf(-alpha * g)) * (u + 1.0f);
   }
+  if (kind == 5) return fmaxf(g, 0.f) * u;
   return gelu_tanh_fast(g) * u;
 }
 
@@ -1200,7 +1201,7 @@ extern "C" int pg_gemm_bf16_fused(const void* x, long long ldx, const void* w, l
   a.tokens = tokens; a.features = features; a.K = K; a.split_k = split_k; a.mode = mode; a.act_gelu = act_gelu;
   a.scale = scale; a.out = out; a.ldo = ldo; a.bias = bias; a.resid = resid; a.ldr = ldr;
   a.glu_alpha = (fu != nullptr && fu->glu_alpha != 0.f) ? fu->glu_alpha : 1.0f;
-  if (mode == PG_EPI_GEGLU && act_gelu != 0 && act_gelu != 1 && act_gelu != 3 && act_gelu != 4) return PG_ERR_ARG;
+  if (mode == PG_EPI_GEGLU && act_gelu != 0 && act_gelu != 1 && act_gelu != 3 && act_gelu != 4 && act_gelu != 5) return PG_ERR_ARG;
   if (fu != nullptr && fu->resid_row_mod > 0) {
     if (swap || resid == nullptr || mode != PG_EPI_F32) return PG_ERR_ARG;  // a token-major fp32 epilogue feature
     a.resid_mod = fu->resid_row_mod;

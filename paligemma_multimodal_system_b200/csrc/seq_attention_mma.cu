@@ -58,7 +58,7 @@ __device__ __forceinline__ void split3(float p, float q, uint32_t& hi, uint32_t&
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-template <int DIM, int VDIM>
+template <int DIM, int VDIM, bool LOGI>
 __global__ void __launch_bounds__(128, (DIM + VDIM <= 128) ? 4 : 2) attn_ragged_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                                                               const bf16* __restrict__ gate, long long ldg, bf16* __restrict__ out,
                                                               const int* __restrict__ entry_row0, const int* __restrict__ entry_n,
@@ -107,6 +107,7 @@ __global__ void __launch_bounds__(128, (DIM + VDIM <= 128) ? 4 : 2) attn_ragged_
   const bool dist = sx.dist_a != nullptr;
   const float da_l = dist ? sx.dist_a[head_l] : 0.f, da_h = dist ? sx.dist_a[head_h] : 0.f;
   const float db_l = dist ? sx.dist_b[head_l] : 0.f, db_h = dist ? sx.dist_b[head_h] : 0.f;
+  const float hb_l = (LOGI && sx.head_bias != nullptr) ? sx.head_bias[head_l] : 0.f, hb_h = (LOGI && sx.head_bias != nullptr) ? sx.head_bias[head_h] : 0.f;
   // key tiles wholly between the kept first keys and the first key inside the window of the CTA's first row are skipped
   const int keep_end = (keep + 63) & ~63;
   const int cta_lo = max(0, ctx + r0 / gsz - window + 1) & ~63;
@@ -164,6 +165,18 @@ __global__ void __launch_bounds__(128, (DIM + VDIM <= 128) ? 4 : 2) attn_ragged_
         mma16816(sacc[nb], qa[ks], b0, b1);
       }
     }
+    if constexpr (LOGI) {
+      // every visible key's weight is the logistic function of its biased score: no maximum, no sum
+#pragma unroll
+      for (int nb = 0; nb < 8; ++nb)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float sc = fmaf(sacc[nb][c], (c & 2) ? sc_h : sc_l, (c & 2) ? hb_h : hb_l);
+          const int away = ((c & 2) ? lim_h : lim_l) - (k0 + nb * 8 + 2 * tq + (c & 1));
+          const bool vis = away >= 0 && (away < window || k0 + nb * 8 + 2 * tq + (c & 1) < keep);
+          sacc[nb][c] = vis ? __fdividef(1.0f, 1.0f + exp2f(sc * -1.4426950408889634f)) : 0.f;
+        }
+    } else {
     // scores -> probabilities (fp32), running max / sum per row; the four lanes of a quad share a row
     float mx_l = -INFINITY, mx_h = -INFINITY;
 #pragma unroll
@@ -203,6 +216,7 @@ __global__ void __launch_bounds__(128, (DIM + VDIM <= 128) ? 4 : 2) attn_ragged_
     for (int nv = 0; nv < NV; ++nv) {
       oacc[nv][0] *= corr_l; oacc[nv][1] *= corr_l; oacc[nv][2] *= corr_h; oacc[nv][3] *= corr_h;
     }
+    }
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
       uint32_t a1[4], a2[4], a3[4];
@@ -228,19 +242,20 @@ __global__ void __launch_bounds__(128, (DIM + VDIM <= 128) ? 4 : 2) attn_ragged_
   }
   l_l += __shfl_xor_sync(0xffffffffu, l_l, 1); l_l += __shfl_xor_sync(0xffffffffu, l_l, 2);
   l_h += __shfl_xor_sync(0xffffffffu, l_h, 1); l_h += __shfl_xor_sync(0xffffffffu, l_h, 2);
+  const long long ldo = sx.out_ld > 0 ? sx.out_ld : (long long)H * VDIM;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int rr = r0 + (half ? rh : rl);
     if (rr >= rows) continue;
     const long long t = row0 + rr / gsz;
     const int head = g * gsz + rr % gsz;
-    float lsum = half ? l_h : l_l, osc = 1.f;
-    if (sx.sink != nullptr) {  // the sink joins the denominator once (m is in base-2 units)
+    float lsum = LOGI ? 1.f : half ? l_h : l_l, osc = 1.f;
+    if (!LOGI && sx.sink != nullptr) {  // the sink joins the denominator once (m is in base-2 units)
       const float mrow = half ? m_h : m_l, sk = sx.sink[head] * 1.4426950408889634f, mm = fmaxf(mrow, sk);
       osc = exp2f(mrow - mm);
       lsum = lsum * osc + exp2f(sk - mm);
     }
-    const float inv = osc / lsum;
+    const float inv = osc / lsum * (sx.out_scale != 0.f ? sx.out_scale : 1.f);
 #pragma unroll
     for (int nv = 0; nv < NV; ++nv) {
       const int col = nv * 8 + 2 * tq;
@@ -252,7 +267,7 @@ __global__ void __launch_bounds__(128, (DIM + VDIM <= 128) ? 4 : 2) attn_ragged_
         v0 *= 1.0f / (1.0f + expf(-gg.x));
         v1 *= 1.0f / (1.0f + expf(-gg.y));
       }
-      *reinterpret_cast<__nv_bfloat162*>(out + t * ((long long)H * VDIM) + (long long)head * VDIM + col) = __floats2bfloat162_rn(v0, v1);
+      *reinterpret_cast<__nv_bfloat162*>(out + t * ldo + (long long)head * VDIM + col) = __floats2bfloat162_rn(v0, v1);
     }
   }
 }
@@ -450,7 +465,7 @@ int launch(const void* q, const void* kp, const void* vp, const void* gate, long
            const int* pt, int max_pages, int page, int entries, int max_n, int H, int G, float scale, float softcap, int skip_single, int gate_per_head,
            const PgAttnScore& sx, cudaStream_t st) {
   const size_t smem = ((size_t)3 * 64 * (DIM + 8) + (size_t)2 * 64 * (VDIM + 8)) * sizeof(bf16);
-  auto kern = attn_ragged_mma_kernel<DIM, VDIM>;
+  auto kern = sx.logistic ? attn_ragged_mma_kernel<DIM, VDIM, true> : attn_ragged_mma_kernel<DIM, VDIM, false>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return PG_ERR_CUDA;
   dim3 grid((max_n * (H / G) + 63) / 64, G, entries);
   kern<<<grid, 128, smem, st>>>(static_cast<const bf16*>(q), static_cast<const bf16*>(kp), static_cast<const bf16*>(vp), static_cast<const bf16*>(gate), ldg,
@@ -468,6 +483,8 @@ extern "C" int pg_attn_ragged_mma(const void* q, const void* k_pages, const void
   if (entries <= 0 || max_n <= 0 || H <= 0 || G <= 0 || (H % G) != 0 || entries > 65535 || G > 65535) return PG_ERR_ARG;
   if (score != nullptr && ((score->dist_a == nullptr) != (score->dist_b == nullptr))) return PG_ERR_ARG;
   const PgAttnScore sx = score != nullptr ? *score : PgAttnScore{};
+  if (sx.logistic && (sx.sink != nullptr || softcap > 0.f || sx.dist_a != nullptr)) return PG_ERR_ARG;  // parts the logistic form is not built with
+  if (sx.out_ld & 1) return PG_ERR_ARG;
   // 16-byte row loads and bf16x2 gate / output accesses
   if (((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_pages) | reinterpret_cast<uintptr_t>(v_pages) | reinterpret_cast<uintptr_t>(out)) & 15) ||
       (gate != nullptr && !gate_per_head && ((reinterpret_cast<uintptr_t>(gate) & 3) || (ldg & 1))))

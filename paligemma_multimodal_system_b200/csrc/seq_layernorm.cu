@@ -4,6 +4,8 @@
 //   pg_layernorm_shift   a = LN(x; w1, b1), b = LN(x; w2, b2) from one mean / variance of the row;
 //                        out1[t] = a[t] + (a[t-1] - a[t]) * shift   (a[-1] = 0; a of a sequence's last token is kept in an
 //                        fp32 state slot, so a portion or a decoded token continues where the sequence stopped), out2[t] = b[t]
+//   pg_gated_layernorm_add  z = y * sigmoid(gate + b), x += LN(z; w1, b1), out = LN(x; w2, b2): the end of a sub-layer whose gated result
+//                        is normalised before it joins the residual, and the input norm of the next one, in one pass over the row
 //   pg_glu               gated-unit activations on a [gate | up] product that the GEMM epilogue did not fuse
 //
 // LN(z) = (z - mean) / sqrt(mean((z - mean)^2) + eps) * w + b, statistics in fp32 from the fp32 residual.
@@ -351,7 +353,7 @@ int launch_ln_vec(const float* x, const float* w1, const float* b1, const float*
   return cudaGetLastError() == cudaSuccess ? PG_OK : PG_ERR_CUDA;
 }
 
-// kind 1: silu(g) * u;  kind 2: g' = min(g, limit), u' = clamp(u, -limit, limit), g' * sigmoid(alpha * g') * (u' + 1)
+// kind 1: silu(g) * u;  kind 3: relu(g) * u;  kind 2: g' = min(g, limit), u' = clamp(u, -limit, limit), g' * sigmoid(alpha * g') * (u' + 1)
 template <typename TA>
 __global__ void glu_kernel(const TA* __restrict__ gu, long long ldgu, TA* __restrict__ out, long long ldo, int F, long long total, int kind,
                            float limit, float alpha) {
@@ -363,6 +365,8 @@ __global__ void glu_kernel(const TA* __restrict__ gu, long long ldgu, TA* __rest
       g = fminf(g, limit);
       u = fminf(fmaxf(u, -limit), limit);
       y = g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+    } else if (kind == 3) {
+      y = fmaxf(g, 0.f) * u;
     } else {
       y = g / (1.0f + expf(-g)) * u;
     }
@@ -370,7 +374,134 @@ __global__ void glu_kernel(const TA* __restrict__ gu, long long ldgu, TA* __rest
   }
 }
 
+// ---------------------------------------------------------------------------------------------------------------------
+// One CTA per row, VT float4 per thread: the row of y, its gate and the residual row are all in flight before the first reduction.
+// ---------------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float4 ld_act4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld_act4(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ float sigmoid1(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+template <typename TA, int VT>
+__global__ void __launch_bounds__(256) gated_layernorm_add_vec_kernel(const float* __restrict__ y, long long ldy, const TA* __restrict__ gate, long long ldg,
+                                                                      const float* __restrict__ gb, const float* __restrict__ w1,
+                                                                      const float* __restrict__ b1, float* __restrict__ x, const float* __restrict__ w2,
+                                                                      const float* __restrict__ b2, TA* __restrict__ out, int D, float eps) {
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 z[VT], r[VT], g[VT];
+#pragma unroll
+  for (int i = 0; i < VT; ++i) {
+    const int d = 4 * (threadIdx.x + 256 * i);
+    const bool ok = d < D;
+    z[i] = ok ? ld4(y + t * ldy + d) : zero;
+    r[i] = ok ? ld4(x + t * D + d) : zero;
+    if (gate != nullptr) g[i] = ok ? ld_act4(gate + t * ldg + d) : zero;
+  }
+  if (gate != nullptr) {
+#pragma unroll
+    for (int i = 0; i < VT; ++i) {
+      const int d = 4 * (threadIdx.x + 256 * i);
+      if (d >= D) continue;
+      const float4 b = ld4(gb + d);
+      z[i].x *= sigmoid1(g[i].x + b.x); z[i].y *= sigmoid1(g[i].y + b.y); z[i].z *= sigmoid1(g[i].z + b.z); z[i].w *= sigmoid1(g[i].w + b.w);
+    }
+  }
+  float mean, rstd;
+  row_stats<VT>(z, D, eps, red, mean, rstd);
+#pragma unroll
+  for (int i = 0; i < VT; ++i) {
+    const int d = 4 * (threadIdx.x + 256 * i);
+    if (d >= D) continue;
+    const float4 a = ln4(z[i], mean, rstd, ld4(w1 + d), ld4(b1 + d));
+    r[i].x += a.x; r[i].y += a.y; r[i].z += a.z; r[i].w += a.w;
+    st4(x + t * D + d, r[i]);
+  }
+  if (out == nullptr) return;
+  row_stats<VT>(r, D, eps, red, mean, rstd);
+#pragma unroll
+  for (int i = 0; i < VT; ++i) {
+    const int d = 4 * (threadIdx.x + 256 * i);
+    if (d < D) st4(out + t * D + d, ln4(r[i], mean, rstd, ld4(w2 + d), ld4(b2 + d)));
+  }
+}
+
+// other widths: the row staged in shared memory
+template <typename TA>
+__global__ void __launch_bounds__(256) gated_layernorm_add_kernel(const float* __restrict__ y, long long ldy, const TA* __restrict__ gate, long long ldg,
+                                                                  const float* __restrict__ gb, const float* __restrict__ w1, const float* __restrict__ b1,
+                                                                  float* __restrict__ x, const float* __restrict__ w2, const float* __restrict__ b2,
+                                                                  TA* __restrict__ out, int D, float eps) {
+  extern __shared__ float buf[];  // [D]; every thread re-reads what it wrote
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  float mean = 0.f, rstd = 0.f;
+  auto stats = [&](float s) {
+    mean = block_sum(s, red) / (float)D;
+    float q = 0.f;
+    for (int d = threadIdx.x; d < D; d += 256) {
+      const float c = buf[d] - mean;
+      q = fmaf(c, c, q);
+    }
+    rstd = 1.0f / sqrtf(block_sum(q, red) / (float)D + eps);
+  };
+  float s = 0.f;
+  for (int d = threadIdx.x; d < D; d += 256) {
+    float v = y[t * ldy + d];
+    if (gate != nullptr) v *= sigmoid1(ld_act(gate, t * ldg + d) + gb[d]);
+    buf[d] = v;
+    s += v;
+  }
+  stats(s);
+  s = 0.f;
+  for (int d = threadIdx.x; d < D; d += 256) {
+    const float v = x[t * D + d] + fmaf((buf[d] - mean) * rstd, w1[d], b1[d]);
+    x[t * D + d] = v;
+    buf[d] = v;
+    s += v;
+  }
+  if (out == nullptr) return;
+  stats(s);
+  for (int d = threadIdx.x; d < D; d += 256) st_act(out, t * D + d, fmaf((buf[d] - mean) * rstd, w2[d], b2[d]));
+}
+
+template <typename TA>
+int launch_gated_ln(const float* y, long long ldy, const void* gate, long long ldg, const float* gb, const float* w1, const float* b1, float* x,
+                    const float* w2, const float* b2, void* out, int rows, int D, float eps, cudaStream_t st) {
+  const TA* g = static_cast<const TA*>(gate);
+  TA* o = static_cast<TA*>(out);
+  auto al = [](const void* p, size_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
+  if (D % 4 == 0 && D <= 8192 && ldy % 4 == 0 && ldg % 4 == 0 && al(y, 16) && al(gate, 4 * sizeof(TA)) && al(gb, 16) && al(w1, 16) && al(b1, 16) && al(x, 16) &&
+      al(w2, 16) && al(b2, 16) && al(out, 4 * sizeof(TA))) {
+#define PG_GLN(VT) gated_layernorm_add_vec_kernel<TA, VT><<<rows, 256, 0, st>>>(y, ldy, g, ldg, gb, w1, b1, x, w2, b2, o, D, eps)
+    if (D <= 1024) PG_GLN(1);
+    else if (D <= 2048) PG_GLN(2);
+    else if (D <= 4096) PG_GLN(4);
+    else PG_GLN(8);
+#undef PG_GLN
+    PG_RET();
+  }
+  const size_t smem = (size_t)D * sizeof(float);
+  if (smem > 200 * 1024) return PG_ERR_ARG;
+  auto kern = gated_layernorm_add_kernel<TA>;
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return PG_ERR_CUDA;
+  kern<<<rows, 256, smem, st>>>(y, ldy, g, ldg, gb, w1, b1, x, w2, b2, o, D, eps);
+  PG_RET();
+}
+
 }  // namespace
+
+extern "C" int pg_gated_layernorm_add(const float* y, long long ldy, const void* gate, long long ldg, const float* gate_b, const float* w1, const float* b1,
+                                      float* x, const float* w2, const float* b2, void* out, int rows, int D, float eps, int act_f32, void* stream) {
+  if (rows <= 0 || D <= 0 || y == nullptr || w1 == nullptr || b1 == nullptr || x == nullptr || (gate != nullptr && gate_b == nullptr) ||
+      (out != nullptr && (w2 == nullptr || b2 == nullptr)))
+    return PG_ERR_ARG;
+  if (act_f32) return launch_gated_ln<float>(y, ldy, gate, ldg, gate_b, w1, b1, x, w2, b2, out, rows, D, eps, PG_ST(stream));
+  return launch_gated_ln<bf16>(y, ldy, gate, ldg, gate_b, w1, b1, x, w2, b2, out, rows, D, eps, PG_ST(stream));
+}
 
 extern "C" int pg_layernorm_shift(const float* x, const float* w1, const float* b1, const float* shift, const float* w2, const float* b2, void* out1,
                                   void* out2, float* state, const int* pos, const int* row_entry, const int* entry_row0, const int* entry_n,
@@ -421,7 +552,7 @@ extern "C" int pg_layernorm_shift(const float* x, const float* w1, const float* 
 
 extern "C" int pg_glu(const void* gu, long long ldgu, void* out, long long ldo, int rows, int F, int kind, float limit, float alpha, int act_f32,
                       void* stream) {
-  if (rows <= 0 || F <= 0 || (kind != 1 && kind != 2)) return PG_ERR_ARG;
+  if (rows <= 0 || F <= 0 || kind < 1 || kind > 3) return PG_ERR_ARG;
   const long long total = (long long)rows * F;
   const int blocks = (int)((total + 255) / 256 < 65535 ? (total + 255) / 256 : 65535);
   if (act_f32)

@@ -5,8 +5,8 @@
 //
 //   pg_attn_prepare        q/k RMS norm (shared per-head weight), interleaved partial rotation, weightless value norm;
 //                          k and v rows go to their cache pages, q to a dense buffer
-//   pg_attn_ragged         causal softmax attention of the new rows over the paged cache (grouped k/v heads, tanh soft cap,
-//                          sigmoid output gate); scores, probabilities and the output accumulation in fp32
+//   pg_attn_ragged         causal softmax (or unnormalised logistic) attention of the new rows over the paged cache (grouped k/v heads,
+//                          tanh soft cap, sigmoid output gate); scores, probabilities and the output accumulation in fp32
 //   pg_linear_attn_scan    decayed outer-product recurrence S <- a S + k v^T, o = S^T q with the state in fp32,
 //                          token by token (decode, short portions)
 //   pg_linear_attn_chunked the same recurrence in blocks of 32 tokens (prompt portions)
@@ -123,7 +123,7 @@ __global__ void __launch_bounds__(128) attn_prepare_kernel(const TA* __restrict_
 // key j for the warp's 4 rows, the warp keeps a running max / sum per row and accumulates P V with lane <-> value columns.
 // VC = ceil(vdim / 32) value columns per lane.
 // ---------------------------------------------------------------------------------------------------------------------
-template <typename TA, int VC>
+template <typename TA, int VC, bool LOGI>
 __global__ void __launch_bounds__(256) attn_ragged_kernel(const TA* __restrict__ q, const TA* __restrict__ k_pages, const TA* __restrict__ v_pages,
                                                           const TA* __restrict__ gate, long long ldg, TA* __restrict__ out,
                                                           const int* __restrict__ entry_row0, const int* __restrict__ entry_n,
@@ -154,7 +154,7 @@ __global__ void __launch_bounds__(256) attn_ragged_kernel(const TA* __restrict__
   }
   float m[4], l[4], o[4][VC];
   int lim[4];  // last visible key of the row = the query's position (-1: row does not exist)
-  float hsc[4], da[4], db[4];  // per-row head constants of the score
+  float hsc[4], da[4], db[4], hb[4];  // per-row head constants of the score
   int wlim = -1;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -168,7 +168,10 @@ __global__ void __launch_bounds__(256) attn_ragged_kernel(const TA* __restrict__
     hsc[i] = scale * (sx.head_scale != nullptr ? sx.head_scale[head] : 1.f);
     da[i] = sx.dist_a != nullptr ? sx.dist_a[head] : 0.f;
     db[i] = sx.dist_a != nullptr ? sx.dist_b[head] : 0.f;
+    hb[i] = (LOGI && sx.head_bias != nullptr) ? sx.head_bias[head] : 0.f;
   }
+  const long long ldo = sx.out_ld > 0 ? sx.out_ld : (long long)H * vdim;
+  const float oscale = sx.out_scale != 0.f ? sx.out_scale : 1.f;
   const int last_row = min(rows, r0 + 32) - 1;
   const int kmax = ctx + last_row / gsz;  // last key any row of this CTA sees
   // first key inside the window of the CTA's / the warp's first row (later rows start later); tiles wholly between the kept first
@@ -217,16 +220,21 @@ __global__ void __launch_bounds__(256) attn_ragged_kernel(const TA* __restrict__
       const bool vis = key <= lim[i] && (lim[i] - key < window || key < keep);
       if (sx.dist_a != nullptr && vis) sc -= da[i] * log1pf(db[i] * (float)(lim[i] - key));
       sc = vis ? sc : -INFINITY;
-      const float mn = fmaxf(m[i], wmax(sc));
-      float pr = 0.f, corr = 1.f;
-      if (mn > -INFINITY) {
-        pr = vis ? expf(sc - mn) : 0.f;
-        corr = expf(m[i] - mn);  // m = -inf on the first visible tile: exp(-inf) = 0
-      }
-      l[i] = l[i] * corr + wsum(pr);
-      m[i] = mn;
+      float pr = 0.f;
+      if (LOGI) {
+        pr = vis ? sigmoidf(sc + hb[i]) : 0.f;
+      } else {
+        const float mn = fmaxf(m[i], wmax(sc));
+        float corr = 1.f;
+        if (mn > -INFINITY) {
+          pr = vis ? expf(sc - mn) : 0.f;
+          corr = expf(m[i] - mn);  // m = -inf on the first visible tile: exp(-inf) = 0
+        }
+        l[i] = l[i] * corr + wsum(pr);
+        m[i] = mn;
 #pragma unroll
-      for (int c = 0; c < VC; ++c) o[i][c] *= corr;
+        for (int c = 0; c < VC; ++c) o[i][c] *= corr;
+      }
       pw[i * 32 + lane] = pr;
     }
     __syncwarp();
@@ -252,11 +260,13 @@ __global__ void __launch_bounds__(256) attn_ragged_kernel(const TA* __restrict__
     if (rr >= rows) continue;
     const long long t = row0 + rr / gsz;
     const int head = g * gsz + rr % gsz;
-    float osc = 1.f;
-    if (sx.sink != nullptr) {  // the sink joins the denominator once; the numerator has no term for it
+    float osc = oscale;
+    if (LOGI) l[i] = 1.f;  // the weights are not normalised
+    if (!LOGI && sx.sink != nullptr) {  // the sink joins the denominator once; the numerator has no term for it
       const float sk = sx.sink[head], mm = fmaxf(m[i], sk);
-      osc = expf(m[i] - mm);
-      l[i] = l[i] * osc + expf(sk - mm);
+      const float f = expf(m[i] - mm);
+      l[i] = l[i] * f + expf(sk - mm);
+      osc *= f;
     }
     const float inv = osc / l[i];
 #pragma unroll
@@ -265,7 +275,7 @@ __global__ void __launch_bounds__(256) attn_ragged_kernel(const TA* __restrict__
       if (col < vdim) {
         float v = o[i][c] * inv;
         if (gate != nullptr) v *= sigmoidf(ldf(gate, t * ldg + (gate_per_head ? (long long)head : (long long)head * vdim + col)));
-        stf(out, t * ((long long)H * vdim) + (long long)head * vdim + col, v);
+        stf(out, t * ldo + (long long)head * vdim + col, v);
       }
     }
   }
@@ -299,7 +309,7 @@ __device__ __forceinline__ void ld8<bf16>(const bf16* p, float* v) {
 // VC = ceil(vdim / 64).  VEC: 16-byte loads -- lane l reads key l's row for the scores; for P V the warp reads four keys per
 // instruction (lane = key l / 8 of the four, value columns 8 (l % 8) .. + 8 of every 64) and the four key groups are summed
 // by shuffles at the end.  All loads of a tile are independent, so a tile costs about one memory round trip.
-template <typename TA, int VC, bool VEC>
+template <typename TA, int VC, bool VEC, bool LOGI>
 __global__ void __launch_bounds__(256) attn_decode_kernel(const TA* __restrict__ q, const TA* __restrict__ k_pages, const TA* __restrict__ v_pages,
                                                           const TA* __restrict__ gate, long long ldg, TA* __restrict__ out, float* __restrict__ partial,
                                                           const int* __restrict__ entry_row0, const int* __restrict__ entry_n,
@@ -325,6 +335,8 @@ __global__ void __launch_bounds__(256) attn_decode_kernel(const TA* __restrict__
     Qs[i] = d < dim ? ldf(q, t * ((long long)H * dim) + (long long)(g * gsz + r) * dim + d) : 0.f;
   }
   __syncthreads();
+  const long long ldo = sx.out_ld > 0 ? sx.out_ld : (long long)H * vdim;
+  const float oscale = sx.out_scale != 0.f ? sx.out_scale : 1.f;
   const int* pt = page_table + (long long)e * max_pages;
   const int ntiles = ctx / 32 + 1;  // keys 0 .. ctx
   // with a window only the tiles of the kept first keys [0, nk) and of the window [t_lo, ntiles) are walked
@@ -335,16 +347,17 @@ __global__ void __launch_bounds__(256) attn_decode_kernel(const TA* __restrict__
   for (int rb = 0; rb < gsz; rb += 4) {
     const int nr = min(4, gsz - rb);
     float m[4], l[4], o[4][NO];
-    float hsc[4], da[4], db[4];
+    float hsc[4], da[4], db[4], hb[4];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      m[i] = -INFINITY; l[i] = 0.f;
+      m[i] = LOGI ? 0.f : -INFINITY; l[i] = 0.f;  // LOGI: a constant maximum, so that partial sums merge with factor one
 #pragma unroll
       for (int c = 0; c < NO; ++c) o[i][c] = 0.f;
       const int head = g * gsz + min(rb + i, gsz - 1);
       hsc[i] = scale * (sx.head_scale != nullptr ? sx.head_scale[head] : 1.f);
       da[i] = sx.dist_a != nullptr ? sx.dist_a[head] : 0.f;
       db[i] = sx.dist_a != nullptr ? sx.dist_b[head] : 0.f;
+      hb[i] = (LOGI && sx.head_bias != nullptr) ? sx.head_bias[head] : 0.f;
     }
     for (int walk = split * 8 + warp; walk < nwalk; walk += nsplit * 8) {
       const int it = walk < nkeep ? walk : t_lo + (walk - nkeep);
@@ -382,13 +395,18 @@ __global__ void __launch_bounds__(256) attn_decode_kernel(const TA* __restrict__
         if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
         if (sx.dist_a != nullptr && vis) sc -= da[i] * log1pf(db[i] * (float)(ctx - j));
         sc = vis ? sc : -INFINITY;
-        const float mn = fmaxf(m[i], wmax(sc));  // every walked tile holds a visible key: mn is finite
-        const float pr = vis ? expf(sc - mn) : 0.f;
-        const float corr = expf(m[i] - mn);
-        l[i] = l[i] * corr + wsum(pr);
-        m[i] = mn;
+        float pr;
+        if (LOGI) {
+          pr = vis ? sigmoidf(sc + hb[i]) : 0.f;
+        } else {
+          const float mn = fmaxf(m[i], wmax(sc));  // every walked tile holds a visible key: mn is finite
+          pr = vis ? expf(sc - mn) : 0.f;
+          const float corr = expf(m[i] - mn);
+          l[i] = l[i] * corr + wsum(pr);
+          m[i] = mn;
 #pragma unroll
-        for (int c = 0; c < NO; ++c) o[i][c] *= corr;
+          for (int c = 0; c < NO; ++c) o[i][c] *= corr;
+        }
         pw[i * 32 + lane] = pr;
       }
       __syncwarp();
@@ -483,14 +501,14 @@ __global__ void __launch_bounds__(256) attn_decode_kernel(const TA* __restrict__
         }
       const int head = g * gsz + rb + i;
       if (nsplit == 1) {
-        if (sx.sink != nullptr) {
+        if (!LOGI && sx.sink != nullptr) {
           const float sk = sx.sink[head], mm = fmaxf(M, sk), f = expf(M - mm);
           acc *= f;
           ls = ls * f + expf(sk - mm);
         }
-        float v = acc / ls;
+        float v = (LOGI ? acc : acc / ls) * oscale;
         if (gate != nullptr) v *= sigmoidf(ldf(gate, t * ldg + (gate_per_head ? (long long)head : (long long)head * vdim + col)));
-        stf(out, t * ((long long)H * vdim) + (long long)head * vdim + col, v);
+        stf(out, t * ldo + (long long)head * vdim + col, v);
       } else {
         float* pp = partial + (((long long)e * H + head) * nsplit + split) * (vdim + 2);
         pp[2 + col] = acc;
@@ -506,7 +524,10 @@ static inline int merge_threads(int vdim) { return vdim <= 64 ? 64 : vdim <= 128
 template <typename TA>
 __global__ void attn_decode_merge_kernel(const float* __restrict__ partial, const TA* __restrict__ gate, long long ldg, TA* __restrict__ out,
                                          const int* __restrict__ entry_row0, const int* __restrict__ entry_n, int H, int vdim, int nsplit,
-                                         int gate_per_head, const float* __restrict__ sink) {
+                                         int gate_per_head, PgAttnScore sx) {
+  const float* sink = sx.logistic ? nullptr : sx.sink;
+  const long long ldo = sx.out_ld > 0 ? sx.out_ld : (long long)H * vdim;
+  const float oscale = sx.out_scale != 0.f ? sx.out_scale : 1.f;
   const int e = blockIdx.y, head = blockIdx.x;
   if (entry_n[e] != 1) return;
   const long long t = entry_row0[e];
@@ -528,9 +549,9 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ partial, cons
       acc *= f;
       ls = ls * f + expf(sk - mm);
     }
-    float v = acc / ls;
+    float v = (sx.logistic ? acc : acc / ls) * oscale;
     if (gate != nullptr) v *= sigmoidf(ldf(gate, t * ldg + (gate_per_head ? (long long)head : (long long)head * vdim + col)));
-    stf(out, t * ((long long)H * vdim) + (long long)head * vdim + col, v);
+    stf(out, t * ldo + (long long)head * vdim + col, v);
   }
 }
 
@@ -803,7 +824,7 @@ static int launch_attn_ragged(const void* q, const void* kp, const void* vp, con
   const int alias = (kp == vp && G == 1 && krow == vrow && vdim <= dim) ? 1 : 0;
   const size_t smem = ((size_t)32 * dimp + 32 * (dimp + 4) + (alias ? 0 : 32 * vdim) + 8 * 128) * sizeof(float);
   if (smem > 220 * 1024) return PG_ERR_ARG;
-  auto kern = attn_ragged_kernel<TA, VC>;
+  auto kern = sx.logistic ? attn_ragged_kernel<TA, VC, true> : attn_ragged_kernel<TA, VC, false>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return PG_ERR_CUDA;
   dim3 grid((max_n * (H / G) + 31) / 32, G, entries);
   kern<<<grid, 256, smem, st>>>(static_cast<const TA*>(q), static_cast<const TA*>(kp), static_cast<const TA*>(vp), static_cast<const TA*>(gate), ldg,
@@ -922,7 +943,7 @@ static int launch_attn_decode(const void* q, const void* kp, const void* vp, con
   const int gsz = H / G, dimp = (dim + 7) & ~7;
   const size_t smem = ((size_t)gsz * dimp + 8 * 128 + 64 + (size_t)32 * vdim) * sizeof(float);
   if (smem > 200 * 1024) return PG_ERR_ARG;
-  auto kern = attn_decode_kernel<TA, VC, VEC>;
+  auto kern = sx.logistic ? attn_decode_kernel<TA, VC, VEC, true> : attn_decode_kernel<TA, VC, VEC, false>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return PG_ERR_CUDA;
   kern<<<dim3(nsplit, G, entries), 256, smem, st>>>(static_cast<const TA*>(q), static_cast<const TA*>(kp), static_cast<const TA*>(vp),
                                                      static_cast<const TA*>(gate), ldg, static_cast<TA*>(out), partial, row0, n, ctx, pt, max_pages, page,
@@ -930,7 +951,7 @@ static int launch_attn_decode(const void* q, const void* kp, const void* vp, con
   pg_count_launch(1);
   if (nsplit > 1) {
     attn_decode_merge_kernel<TA><<<dim3(H, entries), merge_threads(vdim), 0, st>>>(partial, static_cast<const TA*>(gate), ldg, static_cast<TA*>(out), row0, n, H, vdim, nsplit,
-                                                                  gate_per_head, sx.sink);
+                                                                  gate_per_head, sx);
     pg_count_launch(1);
   }
   return cudaGetLastError() == cudaSuccess ? PG_OK : PG_ERR_CUDA;
@@ -940,13 +961,13 @@ extern "C" int pg_attn_decode_merge(const float* partial, const void* gate, long
                                     int entries, int nsplit, int H, int vdim, int gate_per_head, int act_f32, const PgAttnScore* score, void* stream) {
   if (entries <= 0 || entries > 65535 || nsplit <= 0 || H <= 0 || vdim <= 0 || partial == nullptr) return PG_ERR_ARG;
   cudaStream_t st = PG_ST(stream);
-  const float* sink = score != nullptr ? score->sink : nullptr;
+  const PgAttnScore sx = score != nullptr ? *score : PgAttnScore{};
   if (act_f32)
     attn_decode_merge_kernel<float><<<dim3(H, entries), merge_threads(vdim), 0, st>>>(partial, static_cast<const float*>(gate), ldg, static_cast<float*>(out), entry_row0, entry_n,
-                                                                     H, vdim, nsplit, gate_per_head, sink);
+                                                                     H, vdim, nsplit, gate_per_head, sx);
   else
     attn_decode_merge_kernel<bf16><<<dim3(H, entries), merge_threads(vdim), 0, st>>>(partial, static_cast<const bf16*>(gate), ldg, static_cast<bf16*>(out), entry_row0, entry_n, H,
-                                                                    vdim, nsplit, gate_per_head, sink);
+                                                                    vdim, nsplit, gate_per_head, sx);
   PG_RET();
 }
 

@@ -9,13 +9,20 @@
                           a per-head score multiplier, a softmax sink, kept first keys, a per-head sigmoid output gate, keys and
                           values borrowed from an earlier layer's cache
   GegluFeedForward        W_down(gelu_tanh(W_gate h) * W_up h)
-  GluFeedForward          W_down(act(W_gate h) * W_up h) with act = silu, or the clamped form min(g, c) sigmoid(a min(g, c)) (clamp(u) + 1);
+  GluFeedForward          W_down(act(W_gate h) * W_up h) with act = silu or relu, or the clamped form min(g, c) sigmoid(a min(g, c)) (clamp(u) + 1);
                           optional biases
   PolyNormFeedForward     W_down P(W_up h + b) + b, P(z) = a N(z) + b N(z^2) + c N(z^3) + e with N = division by the row's root mean square
   TokenSideInput          a per-layer, per-token low-dimensional embedding gated by a projection of the residual stream
   LatentAttention         attention over ONE cached low-rank row per token (+ one rotated key part shared by the heads); optional, each a
                           parameter: half-split rotation layout, ramped frequency rescaling with a cos / sin gain, a sliding window, a
                           per-element (instead of per-head) sigmoid output gate, cached rows borrowed from an earlier layer
+  ProjectedMixer          base of the sub-layers below: one input projection for everything read from h (and, on request, for rows the caller
+                          adds), a core that maps its columns to the activations of one output projection
+  LogisticAttention       grouped-query attention whose weights are sigmoid(score + bias), not normalised over the keys; half-split rotation
+  ChannelDeltaRule        gated delta rule with one decay per head and key channel behind short convolutions; per-head output norm and gate
+  StateSpaceMixer         scalar-decay state-space recurrence (Mamba-2) behind a short convolution; gate before a grouped output norm
+  MatrixMemory            matrix memory with exponential gates, running maximum and normaliser (mLSTM); per-head output norm and gate
+  SideBySide              two mixers on the same input, a weighted sum of their outputs: joint input and output projections
 
 Every sub-layer gets its weights from a name -> tensor dict (`take(name)` pops and checks the shape), packs them once for a
 `Precision`, says what it keeps per sequence (`cache_spec`), and maps the step's rows h [T, D] (activation type) to
@@ -280,13 +287,15 @@ class GegluFeedForward:
 
 
 class GluFeedForward:
-    """W_down (act(W_gate h) * W_up h) (+ biases).  activation "silu": silu(g) * u; "clamped": g' = min(g, limit),
+    """W_down (act(W_gate h) * W_up h) (+ biases).  activation "silu": silu(g) * u; "relu": relu(g) * u; "clamped": g' = min(g, limit),
     u' = clamp(u, -limit, limit), g' * sigmoid(alpha * g') * (u' + 1)."""
 
     def __init__(self, width, ff, activation="silu", limit=0.0, alpha=1.0, bias=False):
-        if activation not in ("silu", "clamped"):
+        kinds = {"silu": seq_ops.GLU_SILU, "clamped": seq_ops.GLU_CLAMPED, "relu": seq_ops.GLU_RELU}
+        if activation not in kinds:
             raise ValueError(f"unknown gated activation {activation!r}")
-        self.D, self.F, self.kind = int(width), int(ff), seq_ops.GLU_CLAMPED if activation == "clamped" else seq_ops.GLU_SILU
+        self.D, self.F, self.kind = int(width), int(ff), kinds[activation]
+        self.epilogue = {"silu": _lib.GLU_SILU, "clamped": _lib.GLU_CLAMPED, "relu": _lib.GLU_RELU}[activation]
         self.limit, self.alpha, self.bias = float(limit), float(alpha), bool(bias)
 
     def load(self, take, pre):
@@ -300,7 +309,7 @@ class GluFeedForward:
         f32 = dict(device="cuda", dtype=torch.float32)
         self.b_down = w["down_b"].to(**f32).contiguous() if self.bias else None
         # bf16: the tcgen05 GEMM computes the gated unit (and adds the biases) in its epilogue from a [64 gate | 64 up] row-interleaved
-        # weight; F is padded to a multiple of 64 with zero rows (both forms map (0, 0) to 0) and zero columns of the down projection
+        # weight; F is padded to a multiple of 64 with zero rows (every form maps (0, 0) to 0) and zero columns of the down projection
         self.fused = prec.dtype == torch.bfloat16 and D % 8 == 0
         if self.fused:
             Fp = (F + 63) // 64 * 64
@@ -327,7 +336,7 @@ class GluFeedForward:
         T = h.shape[0]
         if self.fused:
             mid = prec.empty(T, self.Fp)
-            _lib.gemm(h, self.w_gu, mid, mode=_lib.EPI_GEGLU, act_gelu=_lib.GLU_CLAMPED if self.kind == seq_ops.GLU_CLAMPED else _lib.GLU_SILU,
+            _lib.gemm(h, self.w_gu, mid, mode=_lib.EPI_GEGLU, act_gelu=self.epilogue,
                       scale=self.limit, glu_alpha=self.alpha, bias=self.b_gu, swap=1 if T <= 128 else 0)
         else:
             gu = seq_ops.linear(h, self.w_gu, prec.empty(T, 2 * self.F), bias=self.b_gu)
@@ -658,3 +667,308 @@ class StreamCoefficients:
             self.read, self.write, self.mix = torch.ones(self.S, **f32), torch.ones(self.S, **f32), torch.eye(self.S, **f32)
         else:
             self.read, self.write, self.mix = (self.w[k].to(**f32).contiguous() for k in ("read", "write", "mix"))
+
+
+# ----------------------------------------------------------------------------------------------------------------------
+# mixers with a joint input projection
+# ----------------------------------------------------------------------------------------------------------------------
+def _pad8(n):
+    return (n + 7) // 8 * 8
+
+
+class ProjectedMixer:
+    """y = W_o core(W_in h).  A mixer names the row blocks of W_in (`in_parts()`: name -> weight, each block starts on a multiple of 8 columns
+    of the product), what it keeps per sequence (`cache_specs()`: a list; the store entries li, li + 1, ... in that order), the width
+    `inner` of its core's output and `core(cols, b, store, li, prec, out)`, which fills out [T, inner] (a view in the activation type)
+    with `out_scale` times its activations.  `pack(prec, side)` appends the rows of `side` to W_in: the mixer then returns (y, side columns),
+    which spares a caller that needs another projection of h a product of its own."""
+
+    out_scale = 1.0
+
+    def pack(self, prec, side=None):
+        parts = dict(self.in_parts())
+        if side is not None:
+            parts["side"] = side
+        self.cols, at = {}, 0
+        for name, w in parts.items():
+            self.cols[name] = (at, at + w.shape[0])
+            at = _pad8(at + w.shape[0])
+        self.w_in = torch.zeros(at, self.D, device="cuda", dtype=prec.dtype)
+        for name, w in parts.items():
+            a, e = self.cols[name]
+            self.w_in[a:e] = w.to("cuda", prec.dtype)
+        self.w_o = self.out_weight().to("cuda", prec.dtype).contiguous()
+        self.pack_core(prec, self.inner)
+
+    def __call__(self, h, b, store, li, prec):
+        proj = seq_ops.linear(h, self.w_in, prec.empty(b.T, self.w_in.shape[0]))
+        cols = {name: proj[:, a:e] for name, (a, e) in self.cols.items()}
+        mid = prec.empty(b.T, self.inner)
+        self.core(cols, b, store, li, prec, mid)
+        y = seq_ops.linear(mid, self.w_o, torch.empty(b.T, self.D, device="cuda", dtype=torch.float32))
+        return (y, cols["side"]) if "side" in cols else y
+
+
+class LogisticAttention(ProjectedMixer):
+    """q = W_q h, k = W_k h, v = W_v h; the first rot_dims dimensions of every q and k head are rotated (element i with element i + rot_dims / 2);
+    out_h(i) = sum over j <= i of sigmoid((q_h(i) . k(j)) * scale + bias_h) v(j)."""
+
+    def __init__(self, width, heads, kv_heads, dim, vdim, scale, rot_dims=0, rot_base=10000.0):
+        if heads % kv_heads:
+            raise ValueError("query heads must be a multiple of key/value heads")
+        if rot_dims % 2 or rot_dims > dim:
+            raise ValueError("rotary dimensions must be even and at most the head size")
+        self.D, self.H, self.G, self.dim, self.vdim = int(width), int(heads), int(kv_heads), int(dim), int(vdim)
+        self.scale, self.rot_dims, self.inner = float(scale), int(rot_dims), int(heads) * int(vdim)
+        self.freq = rotary_frequencies(rot_base, rot_dims) if rot_dims else torch.zeros(1, dtype=torch.float64)
+
+    def cache_specs(self):
+        return [("kv", self.G * self.dim, self.G * self.vdim)]
+
+    def load(self, take, pre):
+        H, G, dim, vdim, D = self.H, self.G, self.dim, self.vdim, self.D
+        self.w = dict(q=take(pre + "q", (H * dim, D)), k=take(pre + "k", (G * dim, D)), v=take(pre + "v", (G * vdim, D)), pb=take(pre + "pb", (H,)),
+                      o=take(pre + "o", (D, H * vdim)))
+
+    def in_parts(self):
+        order = torch.tensor(half_to_pair_order(self.dim, self.rot_dims))  # the rotation kernel turns neighbouring pairs
+
+        def paired(w, n):
+            return w.view(n, self.dim, self.D)[:, order.to(w.device)].reshape(n * self.dim, self.D)
+
+        w = self.w
+        return {"qkv": torch.cat([paired(w["q"], self.H), paired(w["k"], self.G), w["v"]], 0)}
+
+    def out_weight(self):
+        return self.w["o"]
+
+    def pack_core(self, prec, pitch):
+        self.freq_d = self.freq.to("cuda")
+        bias = self.w["pb"].to("cuda", torch.float32).contiguous()
+        self.score = seq_ops.ScoreOptions(self.H, logistic=True, head_bias=bias, out_scale=self.out_scale, out_ld=pitch)
+
+    def core(self, cols, b, store, li, prec, out):
+        H, G, dim, vdim = self.H, self.G, self.dim, self.vdim
+        q = prec.empty(b.T, H * dim)
+        kp, vp = store.k_pages[li], store.v_pages[li]
+        seq_ops.attn_prepare(cols["qkv"], b, self.freq_d, None, None, q, kp, vp, H, G, dim, vdim, self.rot_dims, 1e-6, PAGE, norm_qk=False, norm_v=False)
+        seq_ops.attn_ragged(q, kp, vp, None, out, b, H, G, dim, vdim, self.scale, 0.0, PAGE, score=self.score)
+
+
+def _conv_rows(parts, taps, width):
+    """Tap-major [taps, width] table from [(first channel, [channels, taps] weight)]; channels between the parts stay zero."""
+    t = torch.zeros(taps, width, dtype=torch.float32)
+    for at, w in parts:
+        t[:, at:at + w.shape[0]] = w.float().cpu().t()
+    return t.to("cuda").contiguous()
+
+
+class ChannelDeltaRule(ProjectedMixer):
+    """q = unit(silu(conv(W_q h))) dim^-1/2, k = unit(silu(conv(W_k h))) (kv_heads x dim), v = silu(conv(W_v h)); per head with state S [dim, vdim]
+        S <- g * S (g: one factor per key channel, exp(-exp(A) softplus(W_a2 W_a1 h + c)));  u = sigmoid(W_b h) (v - S^T k);  S <- S + k u^T;
+        out = rms(S^T q) w * sigmoid(W_g2 W_g1 h)
+    (unit divides by the Euclidean norm; the output norm is per head).  The inner width of the two low-rank projections is whatever
+    the checkpoint has."""
+
+    def __init__(self, width, heads, kv_heads, dim, vdim, taps, eps):
+        if heads % kv_heads:
+            raise ValueError("heads must be a multiple of query/key heads")
+        if not 1 <= int(taps) <= 8:
+            raise ValueError("the convolution kernel takes one to eight taps")
+        self.D, self.H, self.G, self.dim, self.vdim, self.taps, self.eps = int(width), int(heads), int(kv_heads), int(dim), int(vdim), int(taps), float(eps)
+        self.inner = self.H * self.vdim
+        self.ck = _pad8(self.G * self.dim)          # first channel of k and of v among the convolution's channels
+        self.cv = 2 * self.ck
+        self.C = self.cv + _pad8(self.H * self.vdim)
+
+    def cache_specs(self):
+        return [("state", (self.H, self.dim, self.vdim)), ("state", (self.taps - 1, self.C)) if self.taps > 1 else None]
+
+    def load(self, take, pre):
+        H, G, dim, vdim, D, K = self.H, self.G, self.dim, self.vdim, self.D, self.taps
+        w = dict(q=take(pre + "q", (G * dim, D)), qc=take(pre + "q.conv", (G * dim, K)), k=take(pre + "k", (G * dim, D)), kc=take(pre + "k.conv", (G * dim, K)),
+                 v=take(pre + "v", (H * vdim, D)), vc=take(pre + "v.conv", (H * vdim, K)), b=take(pre + "b", (H, D)), A_log=take(pre + "A_log", (H,)),
+                 norm=take(pre + "norm", (vdim,)), a1=take(pre + "a1", (None, D)), dt_bias=take(pre + "dt_bias", (H * dim,)), g1=take(pre + "g1", (None, D)),
+                 o=take(pre + "o", (D, H * vdim)))
+        w["a2"] = take(pre + "a2", (H * dim, w["a1"].shape[0]))
+        w["g2"] = take(pre + "g2", (H * vdim, w["g1"].shape[0]))
+        self.w = w
+
+    def in_parts(self):
+        # the low-rank rows are padded to a multiple of 8 with zeros, so that their columns are a whole operand of the second product
+        def padded(t):
+            return torch.cat([t, torch.zeros(_pad8(t.shape[0]) - t.shape[0], self.D, dtype=t.dtype, device=t.device)])
+
+        w = self.w
+        return {"q": w["q"], "k": w["k"], "v": w["v"], "a1": padded(w["a1"]), "g1": padded(w["g1"]), "b": w["b"]}
+
+    def out_weight(self):
+        return self.w["o"]
+
+    def pack_core(self, prec, pitch):
+        w, f32 = self.w, dict(device="cuda", dtype=torch.float32)
+
+        def wide(t):
+            out = torch.zeros(t.shape[0], _pad8(t.shape[1]), device="cuda", dtype=prec.dtype)
+            out[:, :t.shape[1]] = t.to("cuda", prec.dtype)
+            return out
+
+        self.w_a2, self.w_g2 = wide(w["a2"]), wide(w["g2"])
+        self.conv_w = _conv_rows([(0, w["qc"]), (self.ck, w["kc"]), (self.cv, w["vc"])], self.taps, self.C)
+        self.A_log, self.dt_bias, self.norm = (w[k].to(**f32).contiguous() for k in ("A_log", "dt_bias", "norm"))
+        x0 = self.cols["q"][0]
+        run = min(64, self.H * self.vdim)  # values have no norm: any grouping of their channels does
+        self.sections = seq_ops.ConvSections([
+            dict(groups=self.G, size=self.dim, xcol=0, ccol=0, unit=True, scale=self.dim ** -0.5),
+            dict(groups=self.G, size=self.dim, xcol=self.cols["k"][0] - x0, ccol=self.ck, unit=True),
+            dict(groups=-(-self.H * self.vdim // run), size=run, total=self.H * self.vdim, xcol=self.cols["v"][0] - x0, ccol=self.cv)])
+
+    def core(self, cols, b, store, li, prec, out):
+        H, G, dim, vdim, T = self.H, self.G, self.dim, self.vdim, b.T
+        u = prec.empty(T, self.C)
+        inv = torch.empty(T, 2 * G, device="cuda", dtype=torch.float32)
+        seq_ops.short_conv(cols["q"], self.conv_w, store.state[li + 1], u, self.sections, b, inv=inv)
+        decay = seq_ops.linear(cols["a1"], self.w_a2, torch.empty(T, H * dim, device="cuda", dtype=torch.float32))
+        gate = seq_ops.linear(cols["g1"], self.w_g2, prec.empty(T, H * vdim))
+        o = torch.empty(T, H * vdim, device="cuda", dtype=torch.float32)
+        seq_ops.delta_rule(u[:, :G * dim], u[:, self.ck:], u[:, self.cv:], cols["b"], inv, decay, self.A_log, self.dt_bias, store.state[li], o, b, H, G, dim, vdim)
+        seq_ops.group_norm_gate(o, self.norm, gate, out, H, self.eps, seq_ops.GATE_SIGMOID_AFTER, self.out_scale)
+
+
+class StateSpaceMixer(ProjectedMixer):
+    """[z | x | B | C | dt] = W_in h; x, B, C <- silu(conv(.) + bias); per head (group h / (heads / groups) of B and C), dt <- softplus(dt + c):
+        S <- exp(-exp(A) dt) S + dt B x^T;  y = S^T C + D x;   out = rms in norm_groups parts (y * silu(z)) * w."""
+
+    def __init__(self, width, heads, groups, state, vdim, taps, norm_groups, eps):
+        self.D, self.H, self.G, self.N, self.vdim, self.taps = int(width), int(heads), int(groups), int(state), int(vdim), int(taps)
+        self.norm_groups, self.eps, self.inner = int(norm_groups), float(eps), int(heads) * int(vdim)
+        if self.H % self.G:
+            raise ValueError("heads must be a multiple of the B / C groups")
+        if self.inner % self.norm_groups:
+            raise ValueError("the inner width must divide into the norm's groups")
+        if not 1 <= self.taps <= 8:
+            raise ValueError("the convolution kernel takes one to eight taps")
+        self.cB = _pad8(self.inner)
+        self.cC = self.cB + _pad8(self.G * self.N)
+        self.C = self.cC + _pad8(self.G * self.N)
+
+    def cache_specs(self):
+        return [("state", (self.H, self.N, self.vdim)), ("state", (self.taps - 1, self.C)) if self.taps > 1 else None]
+
+    def load(self, take, pre):
+        H, inner, gn = self.H, self.inner, self.G * self.N
+        chans = inner + 2 * gn
+        self.w = {"in": take(pre + "in", (inner + chans + H, self.D)), "conv": take(pre + "conv", (chans, self.taps)), "conv_b": take(pre + "conv.b", (chans,)),
+                  "dt_bias": take(pre + "dt_bias", (H,)), "A_log": take(pre + "A_log", (H,)), "D": take(pre + "D", (H,)), "norm": take(pre + "norm", (inner,)),
+                  "o": take(pre + "o", (self.D, inner))}
+
+    def in_parts(self):
+        z, x, B, C, dt = torch.split(self.w["in"], [self.inner, self.inner, self.G * self.N, self.G * self.N, self.H], 0)
+        return {"z": z, "x": x, "B": B, "C": C, "dt": dt}
+
+    def out_weight(self):
+        return self.w["o"]
+
+    def pack_core(self, prec, pitch):
+        w, f32, inner, gn = self.w, dict(device="cuda", dtype=torch.float32), self.inner, self.G * self.N
+        at = ((0, 0, inner), (self.cB, inner, inner + gn), (self.cC, inner + gn, inner + 2 * gn))
+        self.conv_w = _conv_rows([(c, w["conv"][a:e]) for c, a, e in at], self.taps, self.C)
+        self.conv_b = _conv_rows([(c, w["conv_b"][a:e, None]) for c, a, e in at], 1, self.C).view(-1)
+        self.dt_bias, self.A_log, self.skip, self.norm = (w[k].to(**f32).contiguous() for k in ("dt_bias", "A_log", "D", "norm"))
+        x0 = self.cols["x"][0]
+
+        def section(name, ccol, n):
+            run = min(64, n)
+            return dict(groups=-(-n // run), size=run, total=n, xcol=self.cols[name][0] - x0, ccol=ccol)
+
+        self.sections = seq_ops.ConvSections([section("x", 0, inner), section("B", self.cB, gn), section("C", self.cC, gn)])
+
+    def core(self, cols, b, store, li, prec, out):
+        H, G, N, vdim, T = self.H, self.G, self.N, self.vdim, b.T
+        u = prec.empty(T, self.C)
+        seq_ops.short_conv(cols["x"], self.conv_w, store.state[li + 1], u, self.sections, b, bias=self.conv_b)
+        o = torch.empty(T, self.inner, device="cuda", dtype=torch.float32)
+        seq_ops.gated_recurrence(seq_ops.STATE_SPACE, u[:, self.cC:], u[:, self.cB:], u[:, :self.inner], cols["dt"], None, self.dt_bias, self.A_log, self.skip,
+                                 store.state[li], None, o, b, H, G, N, vdim)
+        seq_ops.group_norm_gate(o, self.norm, cols["z"], out, self.norm_groups, self.eps, seq_ops.GATE_SILU_BEFORE, self.out_scale)
+
+
+class MatrixMemory(ProjectedMixer):
+    """q = W_q h dim^-1/2, k = W_k h, v = W_v h; per head the log gates i = cap tanh((W_i h + b) / cap), f = log sigmoid(cap tanh((W_f h + b) / cap)),
+    the running maximum m' = max(f + m, i) (from 0), and with keep = exp(f + m - m'), put = exp(i - m'):
+        S <- keep S + put k v^T;  n <- keep n + put k;  out = rms(S^T q / (max(|n . q|, exp(-m')) + 1e-6)) w * sigmoid(W_g h)   (norm per head)."""
+
+    def __init__(self, width, heads, dim, vdim, gate_cap, eps):
+        self.D, self.H, self.dim, self.vdim, self.cap, self.eps = int(width), int(heads), int(dim), int(vdim), float(gate_cap), float(eps)
+        self.inner = self.H * self.vdim
+        if not self.cap > 0.0:
+            raise ValueError("the gates' cap must be positive")
+
+    def cache_specs(self):
+        blocks = -(-self.vdim // seq_ops.recurrence_block(self.vdim))
+        return [("state", (self.H, self.dim, self.vdim)), ("state", (blocks, self.H, self.dim + 1))]
+
+    def load(self, take, pre):
+        H, dim, vdim, D = self.H, self.dim, self.vdim, self.D
+        self.w = dict(q=take(pre + "q", (H * dim, D)), k=take(pre + "k", (H * dim, D)), v=take(pre + "v", (H * vdim, D)), g=take(pre + "g", (H * vdim, D)),
+                      o=take(pre + "o", (D, H * vdim)), norm=take(pre + "norm", (H * vdim,)), i=take(pre + "i", (H, D)), ib=take(pre + "i.b", (H,)),
+                      f=take(pre + "f", (H, D)), fb=take(pre + "f.b", (H,)))
+
+    def in_parts(self):
+        return {k: self.w[k] for k in ("q", "k", "v", "g", "i", "f")}
+
+    def out_weight(self):
+        return self.w["o"]
+
+    def pack_core(self, prec, pitch):
+        self.norm, self.ib, self.fb = (self.w[k].to("cuda", torch.float32).contiguous() for k in ("norm", "ib", "fb"))
+
+    def core(self, cols, b, store, li, prec, out):
+        H, dim, vdim = self.H, self.dim, self.vdim
+        o = torch.empty(b.T, self.inner, device="cuda", dtype=torch.float32)
+        seq_ops.gated_recurrence(seq_ops.MATRIX_MEMORY, cols["q"], cols["k"], cols["v"], cols["i"], cols["f"], self.ib, self.fb, None, store.state[li],
+                                 store.state[li + 1], o, b, H, H, dim, vdim, qscale=dim ** -0.5, cap=self.cap)
+        seq_ops.group_norm_gate(o, self.norm, cols["g"], out, H, self.eps, seq_ops.GATE_SIGMOID_AFTER, self.out_scale)
+
+
+class SideBySide(ProjectedMixer):
+    """left_scale * left(h) + right_scale * right(h): one input projection for both mixers, each core fills its columns of one activation row
+    (its scale applied in fp32 there), and one output projection over the joined columns adds the two."""
+
+    def __init__(self, left: ProjectedMixer, right: ProjectedMixer, left_scale=1.0, right_scale=1.0):
+        if left.D != right.D:
+            raise ValueError("both mixers read rows of one width")
+        self.D, self.left, self.right = left.D, left, right
+        left.out_scale, right.out_scale = float(left_scale), float(right_scale)
+        self.at = _pad8(left.inner)
+        self.inner = _pad8(self.at + right.inner)
+
+    def cache_specs(self):
+        return self.left.cache_specs() + self.right.cache_specs()
+
+    def load(self, take, pre):
+        self.left.load(take, pre + "left.")
+        self.right.load(take, pre + "right.")
+
+    def in_parts(self):
+        return {f"{side}.{k}": w for side, mx in (("left", self.left), ("right", self.right)) for k, w in mx.in_parts().items()}
+
+    def out_weight(self):
+        wl, wr = self.left.out_weight(), self.right.out_weight()
+        w = torch.zeros(self.D, self.inner, dtype=wl.dtype, device=wl.device)
+        w[:, :self.left.inner] = wl
+        w[:, self.at:self.at + self.right.inner] = wr
+        return w
+
+    def pack_core(self, prec, pitch):
+        for side, mx in (("left", self.left), ("right", self.right)):
+            mx.cols = {k[len(side) + 1:]: v for k, v in self.cols.items() if k.startswith(side + ".")}
+            mx.pack_core(prec, pitch)
+
+    def core(self, cols, b, store, li, prec, out):
+        if self.at > self.left.inner:
+            out[:, self.left.inner:self.at] = 0  # columns between the parts meet zero weights; they only have to be finite
+        if self.inner > self.at + self.right.inner:
+            out[:, self.at + self.right.inner:] = 0
+        for side, mx, at, base in (("left", self.left, 0, li), ("right", self.right, self.at, li + len(self.left.cache_specs()))):
+            mx.core({k[len(side) + 1:]: v for k, v in cols.items() if k.startswith(side + ".")}, b, store, base, prec, out[:, at:at + mx.inner])

@@ -68,9 +68,15 @@ def _load_zigivik(path, dtype=torch.bfloat16, **kw):
     return load_zigivik(path, dtype)
 
 
+def _load_fadosun(path, dtype=torch.bfloat16, **kw):
+    from .modeling_fadosun import load_fadosun
+    return load_fadosun(path, dtype)
+
+
 for _n in ("paligemma", "PaliGemmaForConditionalGeneration"):
     register(_n, _load_paligemma)
 register("Mapedra", _load_mapedra)
 register("Pukerax", _load_pukerax)
 register("Kovusun", _load_kovusun)
 register("Zigivik", _load_zigivik)
+register("Fadosun", _load_fadosun)

@@ -245,11 +245,11 @@ def sigmoid_gate_mul(y, gate):
     return y
 
 
-GLU_SILU, GLU_CLAMPED = 1, 2
+GLU_SILU, GLU_CLAMPED, GLU_RELU = 1, 2, 3
 
 
 def glu(gu, out, kind, limit=0.0, alpha=1.0):
-    """out[t, f] from the [gate | up] product gu [rows, 2F]: GLU_SILU silu(g) * u; GLU_CLAMPED min(g, limit) * sigmoid(alpha * .) * (clamp(u) + 1)."""
+    """out[t, f] from the [gate | up] product gu [rows, 2F]: GLU_SILU silu(g) * u; GLU_RELU relu(g) * u; GLU_CLAMPED min(g, limit) * sigmoid(alpha * .) * (clamp(u) + 1)."""
     rows, F = out.shape
     assert gu.shape[1] == 2 * F and gu.dtype == out.dtype and gu.stride(1) == 1 and out.stride(1) == 1
     _lib.check(_lib.lib().pg_glu(gu.data_ptr(), gu.stride(0), out.data_ptr(), out.stride(0), rows, F, int(kind), float(limit), float(alpha),
@@ -312,17 +312,25 @@ def attn_prepare(qkv, b: StepBatch, freq, q_norm, k_norm, q_out, k_pages, v_page
 class ScoreOptions:
     """The optional parts of a softmax attention's score and mask, as the kernels read them (PgAttnScore): a sliding window of
     `window` keys (None: all) that keeps the first `keep_first` keys of the sequence visible, a per-head sink logit in the softmax
-    denominator, a penalty dist_a[h] * log(1 + dist_b[h] * distance), a per-head score multiplier.  Tensors: fp32 [H] on the device."""
+    denominator, a penalty dist_a[h] * log(1 + dist_b[h] * distance), a per-head score multiplier.  logistic: no softmax -- a visible
+    key weighs sigmoid(score + head_bias[h]), unnormalised.  out_scale multiplies the output, whose rows are out_ld elements apart
+    (0: dense).  Tensors: fp32 [H] on the device."""
 
-    def __init__(self, heads, window=None, keep_first=0, sink=None, dist_a=None, dist_b=None, head_scale=None):
-        for t in (sink, dist_a, dist_b, head_scale):
+    def __init__(self, heads, window=None, keep_first=0, sink=None, dist_a=None, dist_b=None, head_scale=None, logistic=False, head_bias=None,
+                 out_scale=1.0, out_ld=0):
+        for t in (sink, dist_a, dist_b, head_scale, head_bias):
             assert t is None or (t.is_cuda and t.dtype == torch.float32 and t.is_contiguous() and t.numel() == heads)
         assert (dist_a is None) == (dist_b is None)
         self.window = int(window) if window else 0
         self.keep_first = int(keep_first) if self.window else 0
-        self._keep = (sink, dist_a, dist_b, head_scale)  # the struct holds raw pointers
-        self.window_only = sink is None and dist_a is None and head_scale is None and not self.keep_first  # nothing but a plain sliding window
-        self.c = _lib.AttnScore(self.window, self.keep_first, _lib.ptr(sink), _lib.ptr(dist_a), _lib.ptr(dist_b), _lib.ptr(head_scale))
+        self._keep = (sink, dist_a, dist_b, head_scale, head_bias)  # the struct holds raw pointers
+        assert not logistic or sink is None
+        self.logistic, self.out_scale, self.out_ld = bool(logistic), float(out_scale), int(out_ld)
+        # nothing but a plain sliding window
+        self.window_only = (sink is None and dist_a is None and head_scale is None and not self.keep_first and not logistic and self.out_scale == 1.0
+                            and not self.out_ld)
+        self.c = _lib.AttnScore(self.window, self.keep_first, _lib.ptr(sink), _lib.ptr(dist_a), _lib.ptr(dist_b), _lib.ptr(head_scale), int(self.logistic),
+                                _lib.ptr(head_bias), self.out_scale, self.out_ld)
 
     def visible_keys(self, context):
         """Upper bound of the keys a query at position `context` reads."""
@@ -576,3 +584,108 @@ def linear_attn(qkv, state, decay, out, b: StepBatch, H, dim, vdim, chunked=None
     fn = _lib.lib().pg_linear_attn_chunked if chunked else _lib.lib().pg_linear_attn_scan
     _lib.check(fn(qkv.data_ptr(), qkv.stride(0), state.data_ptr(), decay.data_ptr(), out.data_ptr(), b.row0.data_ptr(), b.n.data_ptr(),
                   b.ctx.data_ptr(), b.slot.data_ptr(), b.E, H, dim, vdim, int(qkv.dtype == torch.float32), _lib.stream()), "pg_linear_attn")
+
+
+# ---- recurrent mixers --------------------------------------------------------------------------------------------------
+def _entry_ptrs(b: StepBatch):
+    return dict(entry_row0=b.row0.data_ptr(), entry_n=b.n.data_ptr(), entry_ctx=b.ctx.data_ptr(), entry_slot=b.slot.data_ptr(), entries=b.E)
+
+
+class ConvSections:
+    """Channel sections of a short convolution: dicts with groups, size (channels of a group), total (channels; default groups * size), xcol
+    (first input column), ccol (first channel of weights, state and output), unit (inverse norms wanted) and scale (factor of the inverse norm)."""
+
+    def __init__(self, sections):
+        assert 1 <= len(sections) <= 3
+        self.c = _lib.ConvSections()
+        self.c.count = len(sections)
+        self.unit_groups = 0
+        for i, s in enumerate(sections):
+            for k in ("groups", "size", "xcol", "ccol"):
+                getattr(self.c, k)[i] = int(s[k])
+            self.c.total[i] = int(s.get("total", s["groups"] * s["size"]))
+            self.c.unit[i] = int(bool(s.get("unit")))
+            self.c.scale[i] = float(s.get("scale", 1.0))
+            if s.get("unit"):
+                self.unit_groups += int(s["groups"])
+
+
+def short_conv(x, w, state, out, sections: ConvSections, b: StepBatch, bias=None, inv=None):
+    """out = silu(causal convolution over time of x's columns, per channel); w fp32 [taps, C] tap-major; state fp32 [slots, taps - 1, C] (None
+    for one tap); inv fp32 [T, unit groups] receives scale / sqrt(sum y^2 + 1e-6) of every group of the unit sections."""
+    import ctypes as C
+    taps, chans = w.shape
+    assert w.dtype == torch.float32 and w.is_contiguous() and x.dtype == out.dtype and x.stride(1) == 1 and out.stride(1) == 1 and out.shape == (b.T, chans)
+    assert taps == 1 or (state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (taps - 1, chans))
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == chans)
+    assert (inv is None) == (sections.unit_groups == 0) and (inv is None or (inv.dtype == torch.float32 and inv.is_contiguous() and inv.shape == (b.T, sections.unit_groups)))
+    _lib.check(_lib.lib().pg_short_conv(x.data_ptr(), x.stride(0), w.data_ptr(), _lib.ptr(bias), _lib.ptr(state), out.data_ptr(), out.stride(0), _lib.ptr(inv),
+                                        sections.unit_groups, C.addressof(sections.c), taps, chans, b.row0.data_ptr(), b.n.data_ptr(), b.ctx.data_ptr(),
+                                        b.slot.data_ptr(), b.E, b.max_n, int(x.dtype == torch.float32), _lib.stream()), "pg_short_conv")
+    return out
+
+
+def recurrence_block(vdim):
+    """Value columns one CTA of the recurrent kernels owns (the normaliser of a matrix memory is kept once per such block)."""
+    return 64 if vdim % 4 == 0 else 16
+
+
+FOREVER = 1 << 30
+
+
+def delta_rule(q, k, v, beta, inv, decay, A_log, dt_bias, state, out, b: StepBatch, H, G, dim, vdim):
+    """Delta rule with a decay per head and key channel (pg_delta_scan): q, k [T, G * dim], v [T, H * vdim], beta [T, H] column views in the
+    activation type, inv fp32 [T, 2 G] (inverse norms of q, then k), decay fp32 [T, H * dim] (before bias and softplus) -> out fp32."""
+    import ctypes as C
+    assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, dim, vdim) and out.dtype == torch.float32 and out.is_contiguous()
+    assert decay.dtype == torch.float32 and decay.stride(1) == 1 and all(t.stride(1) == 1 and t.dtype == q.dtype for t in (q, k, v, beta))
+    a = _lib.DeltaArgs(q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), beta=beta.data_ptr(), ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0),
+                       ldb=beta.stride(0), inv=inv.data_ptr(), ldi=inv.stride(0), decay=decay.data_ptr(), lda=decay.stride(0), A_log=A_log.data_ptr(),
+                       dt_bias=dt_bias.data_ptr(), state=state.data_ptr(), out=out.data_ptr(), H=H, G=G, dim=dim, vdim=vdim, **_entry_ptrs(b))
+    _lib.check(_lib.lib().pg_delta_scan(C.addressof(a), 1, FOREVER, int(q.dtype == torch.float32), _lib.stream()), "pg_delta_scan")
+    return out
+
+
+STATE_SPACE, MATRIX_MEMORY = 0, 1
+
+
+def gated_recurrence(kind, q, k, v, gate1, gate2, p1, p2, p3, state, norm_state, out, b: StepBatch, H, G, dim, vdim, qscale=1.0, cap=0.0):
+    """Recurrence with one scalar decay per head and token (pg_gated_scan; kind STATE_SPACE or MATRIX_MEMORY) -> out fp32 [T, H * vdim]."""
+    import ctypes as C
+    assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, dim, vdim) and out.dtype == torch.float32 and out.is_contiguous()
+    assert all(t is None or (t.stride(1) == 1 and t.dtype == q.dtype) for t in (q, k, v, gate1, gate2)) and (gate2 is None or gate2.stride(0) == gate1.stride(0))
+    if kind == MATRIX_MEMORY:
+        vb = recurrence_block(vdim)
+        assert norm_state.dtype == torch.float32 and tuple(norm_state.shape[1:]) == (-(-vdim // vb), H, dim + 1)
+    a = _lib.GatedArgs(q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0), qscale=float(qscale),
+                       gate1=gate1.data_ptr(), gate2=_lib.ptr(gate2), ldg=gate1.stride(0), p1=p1.data_ptr(), p2=p2.data_ptr(), p3=_lib.ptr(p3), cap=float(cap),
+                       state=state.data_ptr(), norm_state=_lib.ptr(norm_state), out=out.data_ptr(), H=H, G=G, dim=dim, vdim=vdim, **_entry_ptrs(b))
+    _lib.check(_lib.lib().pg_gated_scan(C.addressof(a), int(kind), 1, FOREVER, int(q.dtype == torch.float32), _lib.stream()), "pg_gated_scan")
+    return out
+
+
+GATE_NONE, GATE_SIGMOID_AFTER, GATE_SILU_BEFORE = 0, 1, 2
+
+
+def group_norm_gate(o, w, gate, out, groups, eps, mode, scale=1.0):
+    """out = scale * norm(o) * w * sigmoid(gate) (GATE_SIGMOID_AFTER) or scale * norm(o * silu(gate)) * w (GATE_SILU_BEFORE), the norm in `groups`
+    equal parts of the row; w fp32 [D] or one group's [D / groups]; out may be a column slice."""
+    rows, D = o.shape
+    assert o.dtype == torch.float32 and o.is_contiguous() and w.dtype == torch.float32 and w.is_contiguous() and out.shape == o.shape and out.stride(1) == 1
+    assert gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1)
+    _lib.check(_lib.lib().pg_group_norm_gate(o.data_ptr(), w.data_ptr(), w.numel(), _lib.ptr(gate), 0 if gate is None else gate.stride(0), int(mode),
+                                             out.data_ptr(), out.stride(0), rows, D, int(groups), float(eps), float(scale), int(out.dtype == torch.float32),
+                                             _lib.stream()), "pg_group_norm_gate")
+    return out
+
+
+def gated_layernorm_add(y, gate, gate_b, w1, b1, x, eps, w2=None, b2=None, out=None):
+    """x += LN(y * sigmoid(gate + gate_b); w1, b1) in place (fp32); out (activation type) = LN(x; w2, b2), the next sub-layer's input, when given."""
+    rows, D = x.shape
+    assert y.dtype == torch.float32 and y.shape == x.shape and y.stride(1) == 1 and x.dtype == torch.float32 and x.is_contiguous()
+    assert gate is None or (gate.shape == x.shape and gate.stride(1) == 1 and (out is None or gate.dtype == out.dtype))
+    assert out is None or (out.is_contiguous() and out.shape == x.shape and w2 is not None and b2 is not None)
+    ref = gate if gate is not None else out
+    _lib.check(_lib.lib().pg_gated_layernorm_add(y.data_ptr(), y.stride(0), _lib.ptr(gate), 0 if gate is None else gate.stride(0), _lib.ptr(gate_b),
+                                                 w1.data_ptr(), b1.data_ptr(), x.data_ptr(), _lib.ptr(w2), _lib.ptr(b2), _lib.ptr(out), rows, D, float(eps),
+                                                 int(ref is not None and ref.dtype == torch.float32), _lib.stream()), "pg_gated_layernorm_add")
