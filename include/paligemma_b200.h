@@ -504,6 +504,11 @@ int pg_recurrence_block(int vdim);
 /* Token by token; entries with fewer than n_min or more than n_max new tokens are left alone (another form advances them). */
 int pg_delta_scan(const PgDeltaArgs* args, int n_min, int n_max, int act_f32, void* stream);
 int pg_gated_scan(const PgGatedArgs* args, int kind, int n_min, int n_max, int act_f32, void* stream);
+/* The same recurrences in blocks of tokens on the tensor cores (bf16 activations; every fp32 operand as three bf16 terms), for entries with at
+ * least n_min new tokens; dim <= 128, dim and vdim multiples of 8, 16-byte aligned rows (else PG_ERR_ARG).  pg_delta_blocks: decay ==
+ * args->decay is OVERWRITTEN (cumulative log decays of the entries it advances); scratch: 3072 bytes per (T / 16 + entries + 1) * H. */
+int pg_gated_blocks(const PgGatedArgs* args, int kind, int n_min, void* stream);
+int pg_delta_blocks(const PgDeltaArgs* args, float* decay, void* scratch, int max_n, int n_min, void* stream);
 
 /* out[t, :] = scale * G(o[t, :]) with G a norm in `groups` equal consecutive parts (each divided by its own root mean square) times w and a
  * gate: gate_mode 1 -- norm(o) * w * sigmoid(gate); 2 -- norm(o * silu(gate)) * w; 0 -- no gate.  w_n == D: a weight per column;

@@ -102,6 +102,8 @@ SIGNATURES = {
     "pg_recurrence_block": [i32],
     "pg_delta_scan": [p, i32, i32, i32, p],
     "pg_gated_scan": [p, i32, i32, i32, i32, p],
+    "pg_gated_blocks": [p, i32, i32, p],
+    "pg_delta_blocks": [p, p, p, i32, i32, p],
     "pg_group_norm_gate": [p, p, i32, p, i64, i32, p, i64, i32, i32, i32, f32, f32, i32, p],
     "pg_gated_layernorm_add": [p, i64, p, i64, p, p, p, p, p, p, p, i32, i32, f32, i32, p],
     "pg_glu": [p, i64, p, i64, i32, i32, i32, f32, f32, i32, p],

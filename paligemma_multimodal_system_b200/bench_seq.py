@@ -829,3 +829,203 @@ def run_zigivik(args):
             out[key] = round(out[key], 1)
     print(json.dumps(out), flush=True)
     return out
+
+
+# ----------------------------------------------------------------------------------------------------------------------
+# `bench.py --arch fadosun`: the Fadosun decoder beside the Mapedra decoder (the closest model of the package: a recurrent matrix state on
+# most layers, softmax attention on every fourth, output norms, gated feed-forward) at equal width / heads / k/v heads / head size /
+# feed-forward / depth
+# ----------------------------------------------------------------------------------------------------------------------
+def fadosun_config(width, heads, kv_heads, dim, ff, vocab, layers, taps=4):
+    """Layer types in turn: delta rule, logistic attention beside a state-space recurrence, delta rule, matrix memory; every head `dim` wide."""
+    delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": taps}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 5e5, "dims": dim // 2}}
+    right = {"heads": heads, "groups": kv_heads, "state": dim, "vdim": dim, "conv": taps, "norm_groups": kv_heads}
+    kinds = [{"type": "channel_delta", "mixer": delta}, {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.8, "right_scale": 0.6}},
+             {"type": "channel_delta", "mixer": delta}, {"type": "mlstm", "mixer": {"heads": heads, "dim": dim, "vdim": dim, "gate_cap": 15.0}}]
+    return {"architecture": "Fadosun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [dict(kinds[i % 4], mlp={"kind": "dense", "ff": ff}) for i in range(layers)]}
+
+
+def random_fadosun(cfg, seed=0):
+    from .modeling_fadosun import FadosunConfig, FadosunForCausalLM
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    c = FadosunConfig(cfg)
+    model = FadosunForCausalLM(c, torch.bfloat16)
+
+    def take(name, shape):
+        shape = tuple(c.layers[0]["mixer"].get("dim", 64) if n is None else n for n in shape)  # low-rank projections: one head's width
+        r = torch.randn(shape, device="cuda", generator=g)
+        if name.endswith(("A_log", "dt_bias")):
+            t = torch.rand(shape, device="cuda", generator=g) * 2.5 - 3.0
+        elif name.endswith("f.b"):
+            t = 3.0 + r
+        elif name.endswith("pb"):
+            t = -6.0 + 0.3 * r
+        elif len(shape) == 1:
+            t = 0.1 * r + (0.0 if name.endswith((".b", ".D")) else 1.0)
+        elif name.endswith("conv"):
+            t = 0.5 * r
+        else:
+            t = r * shape[-1] ** -0.5
+        return t.to(torch.bfloat16)
+
+    model.embed = take("embed", (c.vocab, c.width))
+    for blk in model.blocks:
+        blk.load(take)
+    model.final_norm, model.final_norm_b, model.head = take("final.norm", (c.width,)), take("final.norm.b", (c.width,)), take("head", (c.vocab, c.width))
+    model.pack()
+    return model
+
+
+def run_fadosun(args):
+    _lib.require_device()
+    torch.cuda.set_device(0)
+    hbm, tflops, src = peaks()
+    W, H, G, dh, F, V, L = args.width, args.heads, args.kv_heads, args.head_dim, args.ff, args.vocab, args.layers
+    B_pre, S, B_dec, ctx = args.prefill_batch, args.seq_len, args.decode_batch, args.context
+    flush = torch.zeros(64 * 1024 * 1024, device="cuda", dtype=torch.float32)  # 256 MB > L2
+    cfg = fadosun_config(W, H, G, dh, F, V, L)
+    out = {"metric": "fadosun_vs_mapedra_tokens_per_s", "dtype": "bf16", "data": "synthetic", "peaks": src,
+           "config": {"width": W, "heads": H, "kv_heads": G, "head_dim": dh, "ff": F, "vocab": V, "layers": L, "types": [l["type"] for l in cfg["layers"][:4]],
+                      "prefill": [B_pre, S], "decode": [B_dec, ctx], "l2": "256 MB buffer rewritten before every timed launch"}}
+    model = random_fadosun(cfg)
+    eng = _throughput(model, args, flush, V, "fadosun", out)
+    prec, k, store = model.prec, {}, eng.store
+    delta, par, mem = (model.blocks[i].mixer for i in (0, 1, 3))
+    left, right = par.left, par.right
+    at = model.cache_at
+    inner = H * dh
+    blk0 = model.blocks[0]
+    for name, (n_seq, n_new, c0) in {"prefill": (B_pre, S, 0), "decode": (B_dec, 1, ctx)}.items():
+        b = _entries(store, n_seq, n_new, c0)
+        T = b.T
+        for t in store.state:
+            if t is not None:
+                t.normal_()
+        x, a = torch.randn(T, W, device="cuda"), prec.empty(T, W)
+        y, gl = torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda").to(torch.bfloat16)
+        s1, s2 = blk0.sub1, blk0.sub2
+        k[f"gated_norm_residual_norm_{name}"] = dict(
+            s=timed(lambda: seq_ops.gated_layernorm_add(y, gl, s1.rg_b, s1.post, s1.post_b, x, 1e-6, s2.pre, s2.pre_b, a), flush=flush), bytes=T * W * (4 + 2 + 8 + 2))
+        h = torch.randn(T, W, device="cuda").to(torch.bfloat16)
+        k[f"feed_forward_{name}"] = dict(s=timed(lambda: blk0.ff(h, b, prec), flush=flush), flops=6 * T * W * F, bytes=3 * W * F * 2 + T * (W * 2 + F * 4 + W * 4))
+        state_rw = n_seq * H * dh * dh * 4 * 2
+        o = torch.empty(T, inner, device="cuda")
+        # delta rule
+        proj = torch.randn(T, delta.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        cols = {n: proj[:, i:j] for n, (i, j) in delta.cols.items()}
+        u, inv = prec.empty(T, delta.C), torch.empty(T, 2 * delta.G, device="cuda")
+        k[f"delta_convolution_{name}"] = dict(
+            s=timed(lambda: seq_ops.short_conv(cols["q"], delta.conv_w, store.state[at[0] + 1], u, delta.sections, b, inv=inv), flush=flush),
+            bytes=T * delta.C * 4 + (n_seq * 3 * delta.C * 8))
+        decay = torch.randn(T, inner, device="cuda") * 0.5
+        k[f"delta_rule_{name}"] = dict(
+            s=timed(lambda: seq_ops.delta_rule(u[:, :delta.G * dh], u[:, delta.ck:], u[:, delta.cv:], cols["b"], inv, decay, delta.A_log, delta.dt_bias,
+                                               store.state[at[0]], o, b, H, delta.G, dh, dh), flush=flush),
+            flops=T * H * 6 * dh * dh, bytes=state_rw + T * inner * (6 + 4 + 4))
+        gate, mid = torch.randn(T, inner, device="cuda").to(torch.bfloat16), prec.empty(T, inner)
+        k[f"head_norm_gate_{name}"] = dict(s=timed(lambda: seq_ops.group_norm_gate(o, delta.norm, gate, mid, H, 1e-6, seq_ops.GATE_SIGMOID_AFTER), flush=flush),
+                                           bytes=T * inner * (4 + 2 + 2))
+        # state space beside logistic attention
+        us = prec.empty(T, right.C)
+        projp = torch.randn(T, par.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        pc = {n: projp[:, i:j] for n, (i, j) in par.cols.items()}
+        k[f"state_space_convolution_{name}"] = dict(
+            s=timed(lambda: seq_ops.short_conv(pc["right.x"], right.conv_w, store.state[at[1] + 2], us, right.sections, b, bias=right.conv_b), flush=flush),
+            bytes=T * right.C * 4 + (n_seq * 3 * right.C * 8))
+        k[f"state_space_{name}"] = dict(
+            s=timed(lambda: seq_ops.gated_recurrence(seq_ops.STATE_SPACE, us[:, right.cC:], us[:, right.cB:], us[:, :inner], pc["right.dt"], None, right.dt_bias,
+                                                     right.A_log, right.skip, store.state[at[1] + 1], None, o, b, H, right.G, dh, dh), flush=flush),
+            flops=T * H * 4 * dh * dh, bytes=state_rw + T * (inner * (2 + 4) + 2 * right.G * dh * 2))
+        k[f"gated_group_norm_{name}"] = dict(
+            s=timed(lambda: seq_ops.group_norm_gate(o, right.norm, pc["right.z"], mid, right.norm_groups, 1e-6, seq_ops.GATE_SILU_BEFORE), flush=flush),
+            bytes=T * inner * (4 + 2 + 2))
+        kp, vp = store.k_pages[at[1]], store.v_pages[at[1]]
+        kp.normal_()
+        vp.normal_()
+        q, both = prec.empty(T, inner), prec.empty(T, par.inner)
+        k[f"attn_prepare_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_prepare(pc["left.qkv"], b, left.freq_d, None, None, q, kp, vp, H, G, dh, dh, left.rot_dims, 1e-6, PAGE, norm_qk=False,
+                                                 norm_v=False), flush=flush), bytes=T * (H + 2 * G) * dh * 2 * 2)
+        pairs = n_seq * (n_new * c0 + n_new * (n_new + 1) // 2)
+        k[f"logistic_attention_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_ragged(q, kp, vp, None, both, b, H, G, dh, dh, left.scale, 0.0, PAGE, score=left.score), flush=flush),
+            flops=4 * dh * H * pairs, bytes=n_seq * (c0 + n_new) * G * 2 * dh * 2 + 2 * T * inner * 2)
+        # matrix memory
+        projm = torch.randn(T, mem.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        mc = {n: projm[:, i:j] for n, (i, j) in mem.cols.items()}
+        store.state[at[3] + 1].fill_(0.5)
+        k[f"matrix_memory_{name}"] = dict(
+            s=timed(lambda: seq_ops.gated_recurrence(seq_ops.MATRIX_MEMORY, mc["q"], mc["k"], mc["v"], mc["i"], mc["f"], mem.ib, mem.fb, None, store.state[at[3]],
+                                                     store.state[at[3] + 1], o, b, H, H, dh, dh, qscale=dh ** -0.5, cap=mem.cap), flush=flush),
+            flops=T * H * 4 * dh * dh, bytes=state_rw + T * inner * (6 + 4))
+        for li, blk in enumerate(model.blocks[:4]):
+            if li == 2:
+                continue
+            mx = blk.mixer
+            k[f"mixer_{cfg['layers'][li]['type']}_{name}"] = dict(
+                s=timed(lambda: mx(h, b, store, at[li], prec), flush=flush), flops=2 * T * W * (mx.w_in.shape[0] + mx.inner),
+                bytes=(mx.w_in.numel() + mx.w_o.numel()) * 2 + T * W * 6 + state_rw)
+        for i in range(n_seq):
+            store.release(("k", i))
+    del eng, model, store
+    torch.cuda.empty_cache()
+
+    # ---------------------------------------------------------------- Mapedra at equal size
+    mm = random_mapedra(mapedra_config(W, H, G, dh, F, V, L))
+    eng = _throughput(mm, args, flush, V, "mapedra", out)
+    store, prec = eng.store, mm.prec
+    li_att = next(i for i, b in enumerate(mm.blocks) if hasattr(b.mixer, "G"))
+    li_lin = next(i for i, b in enumerate(mm.blocks) if hasattr(b.mixer, "decay"))
+    att, lin = mm.blocks[li_att].mixer, mm.blocks[li_lin].mixer
+    for name, (n_seq, n_new, c0) in {"prefill": (B_pre, S, 0), "decode": (B_dec, 1, ctx)}.items():
+        b = _entries(store, n_seq, n_new, c0)
+        T = b.T
+        proj = torch.randn(T, att.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        q, o = prec.empty(T, inner), prec.empty(T, inner)
+        kp, vp = store.k_pages[li_att], store.v_pages[li_att]
+        kp.normal_()
+        vp.normal_()
+        gate = proj[:, (H + G) * dh + G * dh:]
+        k[f"mapedra_attn_prepare_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_prepare(proj, b, att.freq_d, att.qn, att.kn, q, kp, vp, H, G, dh, dh, att.rot_dims, 1e-6, PAGE), flush=flush),
+            bytes=T * (H + 2 * G) * dh * 2 * 2)
+        pairs = n_seq * (n_new * c0 + n_new * (n_new + 1) // 2)
+        k[f"mapedra_attention_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_ragged(q, kp, vp, gate, o, b, H, G, dh, dh, att.scale, att.softcap, PAGE), flush=flush),
+            flops=4 * dh * H * pairs, bytes=n_seq * (c0 + n_new) * G * 2 * dh * 2 + 3 * T * inner * 2)
+        projl = torch.randn(T, lin.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        ol = torch.empty(T, inner, device="cuda", dtype=torch.float32)
+        k[f"mapedra_lightning_{name}"] = dict(
+            s=timed(lambda: seq_ops.linear_attn(projl, store.state[li_lin], lin.decay_d, ol, b, H, dh, dh), flush=flush),
+            flops=T * H * 4 * dh * dh, bytes=n_seq * H * dh * dh * 4 * 2 + T * inner * (3 * 2 + 4))
+        attl = prec.empty(T, inner)
+        k[f"mapedra_lightning_norm_gate_{name}"] = dict(
+            s=timed(lambda: seq_ops.rmsnorm_gate(ol, lin.norm, projl[:, 3 * inner:], attl, 1e-6), flush=flush), bytes=T * inner * (4 + 2 + 2))
+        y, x, xa = torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda"), prec.empty(T, W)
+        w1 = torch.ones(W, device="cuda")
+        k[f"mapedra_group_norm_residual_{name}"] = dict(s=timed(lambda: seq_ops.group_rmsnorm_add(y, w1, x, xa, 4, 1e-6), flush=flush), bytes=T * W * (4 + 8 + 2))
+        h = torch.randn(T, W, device="cuda").to(torch.bfloat16)
+        ffm = mm.blocks[0].ff
+        k[f"mapedra_geglu_feed_forward_{name}"] = dict(s=timed(lambda: ffm(h, b, prec), flush=flush), flops=6 * T * W * ffm.F,
+                                                       bytes=3 * W * ffm.F * 2 + T * (W * 2 + ffm.F * 4 + W * 4))
+        for i in range(n_seq):
+            store.release(("k", i))
+    for name, d in k.items():
+        d["us"] = round(d.pop("s") * 1e6, 2)
+        d["hbm_frac"] = round(d["bytes"] / (d["us"] * 1e-6) / hbm, 4)
+        if "flops" in d:
+            d["tflops"] = round(d["flops"] / (d["us"] * 1e-6) / 1e12, 2)
+            d["tensor_frac"] = round(d["flops"] / (d["us"] * 1e-6) / tflops, 5)
+        bound = max(d["bytes"] / hbm, d.get("flops", 0) / tflops)
+        d["x_roofline"] = round(d["us"] * 1e-6 / bound, 2)
+    out["kernels"] = k
+    out["value"] = out["fadosun_decode_tok_s"]
+    out["unit"] = "tokens/s"
+    out["n_gpus"] = 1
+    for key in list(out):
+        if key.endswith("tok_s"):
+            out[key] = round(out[key], 1)
+    print(json.dumps(out), flush=True)
+    return out

@@ -14,10 +14,8 @@ INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 LIB = os.path.join(HERE, "libpaligemma_b200.so")
 OBJ_DIR = os.path.join(HERE, "build")
 
-NVCC_FLAGS = [
-    "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
-    "-Xcompiler", "-fPIC", "-I", INCLUDE, "-I", CSRC,
-]
+CODE_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC"]
+NVCC_FLAGS = CODE_FLAGS + ["-I", INCLUDE, "-I", CSRC]  # the include paths are not part of the stamps: a built checkout may be moved
 
 
 def _sources():
@@ -32,7 +30,7 @@ def _stamp():
                 with open(os.path.join(root, f), "rb") as fh:
                     h.update(f.encode())
                     h.update(fh.read())
-    h.update(" ".join(NVCC_FLAGS).encode())
+    h.update(" ".join(CODE_FLAGS).encode())
     return h.hexdigest()
 
 
@@ -56,7 +54,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
         obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
         h = headers.copy()
         h.update(open(src, "rb").read())
-        h.update(" ".join(NVCC_FLAGS).encode())
+        h.update(" ".join(CODE_FLAGS).encode())
         mark = obj + ".stamp"
         if not force and not verbose and os.path.exists(obj) and os.path.exists(mark) and open(mark).read() == h.hexdigest():
             return obj

@@ -630,11 +630,23 @@ def recurrence_block(vdim):
     return 64 if vdim % 4 == 0 else 16
 
 
+# an entry with at least this many new tokens is advanced in blocks on the tensor cores (bf16, head sizes that are multiples of 8 up to 128),
+# anything else token by token; the form an entry takes depends on its own length only
+RECURRENCE_BLOCK_MIN = 16
 FOREVER = 1 << 30
 
 
-def delta_rule(q, k, v, beta, inv, decay, A_log, dt_bias, state, out, b: StepBatch, H, G, dim, vdim):
-    """Delta rule with a decay per head and key channel (pg_delta_scan): q, k [T, G * dim], v [T, H * vdim], beta [T, H] column views in the
+def _in_blocks(q, k, v, dim, vdim, b: StepBatch, blocks):
+    """None: token by token; else the least number of new tokens that goes through the block kernels."""
+    fits = (q.dtype == torch.bfloat16 and dim % 8 == 0 and dim <= 128 and vdim % 8 == 0
+            and all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v)))
+    n_min = RECURRENCE_BLOCK_MIN if blocks is None else (1 if blocks else FOREVER)
+    return n_min if fits and b.max_n >= n_min else None
+
+
+def delta_rule(q, k, v, beta, inv, decay, A_log, dt_bias, state, out, b: StepBatch, H, G, dim, vdim, blocks=None):
+    """Delta rule with a decay per head and key channel (pg_delta_blocks / pg_delta_scan; blocks True / False: one form for every entry that fits
+    it; `decay` is scratch afterwards): q, k [T, G * dim], v [T, H * vdim], beta [T, H] column views in the
     activation type, inv fp32 [T, 2 G] (inverse norms of q, then k), decay fp32 [T, H * dim] (before bias and softplus) -> out fp32."""
     import ctypes as C
     assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, dim, vdim) and out.dtype == torch.float32 and out.is_contiguous()
@@ -642,15 +654,23 @@ def delta_rule(q, k, v, beta, inv, decay, A_log, dt_bias, state, out, b: StepBat
     a = _lib.DeltaArgs(q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), beta=beta.data_ptr(), ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0),
                        ldb=beta.stride(0), inv=inv.data_ptr(), ldi=inv.stride(0), decay=decay.data_ptr(), lda=decay.stride(0), A_log=A_log.data_ptr(),
                        dt_bias=dt_bias.data_ptr(), state=state.data_ptr(), out=out.data_ptr(), H=H, G=G, dim=dim, vdim=vdim, **_entry_ptrs(b))
-    _lib.check(_lib.lib().pg_delta_scan(C.addressof(a), 1, FOREVER, int(q.dtype == torch.float32), _lib.stream()), "pg_delta_scan")
+    n_min = _in_blocks(q, k, v, dim, vdim, b, blocks) if decay.stride(0) % 4 == 0 else None
+    if n_min is not None:
+        scratch = torch.empty((b.T // 16 + b.E + 1) * H * 192, 4, device="cuda", dtype=torch.int32)
+        _lib.check(_lib.lib().pg_delta_blocks(C.addressof(a), decay.data_ptr(), scratch.data_ptr(), b.max_n, n_min, _lib.stream()), "pg_delta_blocks")
+    if n_min is None or (n_min > 1 and b.E > 1):
+        _lib.check(_lib.lib().pg_delta_scan(C.addressof(a), 1, FOREVER if n_min is None else n_min - 1, int(q.dtype == torch.float32), _lib.stream()),
+                   "pg_delta_scan")
     return out
 
 
 STATE_SPACE, MATRIX_MEMORY = 0, 1
 
 
-def gated_recurrence(kind, q, k, v, gate1, gate2, p1, p2, p3, state, norm_state, out, b: StepBatch, H, G, dim, vdim, qscale=1.0, cap=0.0):
-    """Recurrence with one scalar decay per head and token (pg_gated_scan; kind STATE_SPACE or MATRIX_MEMORY) -> out fp32 [T, H * vdim]."""
+def gated_recurrence(kind, q, k, v, gate1, gate2, p1, p2, p3, state, norm_state, out, b: StepBatch, H, G, dim, vdim, qscale=1.0, cap=0.0,
+                     blocks=None):
+    """Recurrence with one scalar decay per head and token (pg_gated_blocks / pg_gated_scan, `blocks` as in delta_rule; kind STATE_SPACE or
+    MATRIX_MEMORY) -> out fp32 [T, H * vdim]."""
     import ctypes as C
     assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, dim, vdim) and out.dtype == torch.float32 and out.is_contiguous()
     assert all(t is None or (t.stride(1) == 1 and t.dtype == q.dtype) for t in (q, k, v, gate1, gate2)) and (gate2 is None or gate2.stride(0) == gate1.stride(0))
@@ -660,7 +680,12 @@ def gated_recurrence(kind, q, k, v, gate1, gate2, p1, p2, p3, state, norm_state,
     a = _lib.GatedArgs(q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0), qscale=float(qscale),
                        gate1=gate1.data_ptr(), gate2=_lib.ptr(gate2), ldg=gate1.stride(0), p1=p1.data_ptr(), p2=p2.data_ptr(), p3=_lib.ptr(p3), cap=float(cap),
                        state=state.data_ptr(), norm_state=_lib.ptr(norm_state), out=out.data_ptr(), H=H, G=G, dim=dim, vdim=vdim, **_entry_ptrs(b))
-    _lib.check(_lib.lib().pg_gated_scan(C.addressof(a), int(kind), 1, FOREVER, int(q.dtype == torch.float32), _lib.stream()), "pg_gated_scan")
+    n_min = _in_blocks(q, k, v, dim, vdim, b, blocks)
+    if n_min is not None:
+        _lib.check(_lib.lib().pg_gated_blocks(C.addressof(a), int(kind), n_min, _lib.stream()), "pg_gated_blocks")
+    if n_min is None or (n_min > 1 and b.E > 1):
+        _lib.check(_lib.lib().pg_gated_scan(C.addressof(a), int(kind), 1, FOREVER if n_min is None else n_min - 1, int(q.dtype == torch.float32),
+                                            _lib.stream()), "pg_gated_scan")
     return out
 
 
