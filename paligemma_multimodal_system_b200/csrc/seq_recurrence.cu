@@ -203,6 +203,108 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const TA* __restrict__ 
   }
 }
 
+// The same for groups of 8 * 2^k <= 256 channels and 16-byte aligned rows (bf16): lane <-> 8 adjacent channels, so that a warp covers 256 adjacent
+// channels of a row (several groups), and the next ROWS_AHEAD rows are in flight while the current one is computed.
+__device__ __forceinline__ void unpack8(uint4 u, float* v) {
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(w[i] << 16);
+    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
+
+template <int TAPS>
+__global__ void __launch_bounds__(128) short_conv_vec_kernel(const bf16* __restrict__ x, long long ldx, const float* __restrict__ w,
+                                                             const float* __restrict__ bias, float* __restrict__ state, bf16* __restrict__ out,
+                                                             long long ldo, float* __restrict__ inv, int ldi, PgConvSections sec, int taps, int C,
+                                                             const int* __restrict__ entry_row0, const int* __restrict__ entry_n,
+                                                             const int* __restrict__ entry_ctx, const int* __restrict__ entry_slot, int chunk) {
+  constexpr int AHEAD = 4;
+  const int e = blockIdx.z, lane = threadIdx.x & 31;
+  const int n = entry_n[e], r0 = blockIdx.y * chunk;
+  if (r0 >= n) return;
+  int g = blockIdx.x * 4 + (threadIdx.x >> 5), s = 0, unit_base = 0;
+  while (s < sec.count && g >= (sec.total[s] + 255) / 256) {
+    g -= (sec.total[s] + 255) / 256;
+    if (sec.unit[s]) unit_base += sec.groups[s];
+    ++s;
+  }
+  if (s >= sec.count) return;
+  const int c = g * 256 + lane * 8;  // channel inside the section
+  const bool ok = c < sec.total[s];  // totals are multiples of 8
+  const int lanes = sec.size[s] / 8; // lanes of one group
+  const long long row0 = entry_row0[e];
+  const bf16* xp = x + row0 * ldx + sec.xcol[s] + (ok ? c : 0);
+  bf16* op = out + row0 * ldo + sec.ccol[s] + (ok ? c : 0);
+  const int cc = sec.ccol[s] + (ok ? c : 0), K = taps - 1;
+  float* slot = state + (long long)entry_slot[e] * K * C + cc;
+  float wt[TAPS][8], bs[8], hist[TAPS - 1][8];
+  auto ld8 = [](const float* p, float* v) { ldv<4>(p, 0, v); ldv<4>(p, 4, v + 4); };
+  auto zero8 = [](float* v) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = 0.f;
+  };
+  if (bias != nullptr) ld8(bias + cc, bs); else zero8(bs);
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+    const int tj = j - (TAPS - taps);
+    if (tj >= 0) ld8(w + (long long)tj * C + cc, wt[j]); else zero8(wt[j]);
+  }
+#pragma unroll
+  for (int j = 0; j < TAPS - 1; ++j) {
+    const int row = r0 - (TAPS - 1) + j;
+    if (row >= 0) unpack8(*reinterpret_cast<const uint4*>(xp + row * ldx), hist[j]);
+    else if (entry_ctx[e] > 0 && K + row >= 0) ld8(slot + (long long)(K + row) * C, hist[j]);
+    else zero8(hist[j]);
+  }
+  const int r1 = min(n, r0 + chunk);
+  uint4 nxt[AHEAD];
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i) nxt[i] = r0 + i < r1 ? *reinterpret_cast<const uint4*>(xp + (long long)(r0 + i) * ldx) : make_uint4(0, 0, 0, 0);
+  for (int rb = r0; rb < r1; rb += AHEAD) {
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      const int r = rb + i;
+      if (r >= r1) break;
+      float cur[8], y[8], ss = 0.f;
+      unpack8(nxt[i], cur);
+      if (r + AHEAD < r1) nxt[i] = *reinterpret_cast<const uint4*>(xp + (long long)(r + AHEAD) * ldx);
+#pragma unroll
+      for (int v = 0; v < 8; ++v) {
+        float a = bs[v];
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) a = fmaf(wt[j][v], hist[j][v], a);
+        a = fmaf(wt[TAPS - 1][v], cur[v], a);
+#pragma unroll
+        for (int j = 0; j < TAPS - 2; ++j) hist[j][v] = hist[j + 1][v];
+        hist[TAPS - 2][v] = cur[v];
+        y[v] = __fdividef(a, 1.0f + __expf(-a));  // a bf16 activation: the hardware exponential is far below its rounding
+      }
+      const uint4 pk = make_uint4(pg::pack_bf16(y[0], y[1]), pg::pack_bf16(y[2], y[3]), pg::pack_bf16(y[4], y[5]), pg::pack_bf16(y[6], y[7]));
+      if (ok) *reinterpret_cast<uint4*>(op + (long long)r * ldo) = pk;
+      if (sec.unit[s]) {
+        unpack8(pk, y);  // the norm is that of the stored activations
+#pragma unroll
+        for (int v = 0; v < 8; ++v) ss = fmaf(y[v], y[v], ss);
+        for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (ok && (lane & (lanes - 1)) == 0) inv[(row0 + r) * ldi + unit_base + c / sec.size[s]] = sec.scale[s] / sqrtf(ss + 1e-6f);
+      }
+    }
+  }
+  if (r0 == 0 && K > 0 && ok) {  // owner of the slot: it becomes the inputs of the entry's last K rows
+    for (int j = 0; j < K; ++j) {
+      const int row = n - K + j;
+      float h[8];
+      if (row >= 0) unpack8(*reinterpret_cast<const uint4*>(xp + (long long)row * ldx), h);
+      else if (entry_ctx[e] > 0) ld8(slot + (long long)(n + j) * C, h);
+      else zero8(h);
+      stv<4>(slot, (long long)j * C, h);
+      stv<4>(slot, (long long)j * C + 4, h + 4);
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------------------
 // Scans.  CTA = (block of 16 * VEC value columns, head, entry); thread = VEC value columns (ct) x every 16th key dimension (grp), its
 // part of the state in registers.  Per token the key-side vectors go through shared memory (double-buffered) and the sums
@@ -494,6 +596,56 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
   }
 }
 
+// Groups of 4 * NV * 2^k columns whose lanes fit a warp: lane <-> NV float4 of one group, several groups per warp, the row read once.
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+
+template <typename TA, int NV>
+__global__ void __launch_bounds__(256) group_norm_gate_flat_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_n,
+                                                                   const TA* __restrict__ gate, long long ldg, int gate_mode, TA* __restrict__ out,
+                                                                   long long ldo, int D, int gs, long long total_groups, float eps, float scale) {
+  const int lanes = gs / (4 * NV), groups = D / gs;
+  const long long id = (long long)blockIdx.x * (256 / lanes) + threadIdx.x / lanes;  // (row, group)
+  const int l = threadIdx.x & (lanes - 1);
+  const bool ok = id < total_groups;
+  const long long t = ok ? id / groups : 0;
+  const int col0 = (ok ? (int)(id % groups) : 0) * gs;
+  float v[NV][4], z[NV][4], s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = col0 + (i * lanes + l) * 4;
+    if (ok) {
+      ldv<4>(o, t * D + d, v[i]);
+      if (gate_mode != 0) ldv<4>(gate, t * ldg + d, z[i]);
+    } else {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[i][k] = z[i][k] = 0.f;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      if (gate_mode != 0) {
+        const float sg = sizeof(TA) == 2 ? fast_sigmoid(z[i][k]) : sigmoid(z[i][k]);
+        if (gate_mode == 2) v[i][k] *= z[i][k] * sg;
+        z[i][k] = sg;
+      }
+      s = fmaf(v[i][k], v[i][k], s);
+    }
+  for (int x = lanes / 2; x > 0; x >>= 1) s += __shfl_xor_sync(0xffffffffu, s, x);
+  if (!ok) return;
+  const float iv = scale / sqrtf(s / (float)gs + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int in = (i * lanes + l) * 4;
+    float ww[4];
+    ldv<4>(w, w_n == gs ? in : col0 + in, ww);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) v[i][k] *= iv * ww[k] * (gate_mode == 1 ? z[i][k] : 1.0f);
+    stv<4>(out, t * ldo + col0 + in, v[i]);
+  }
+}
+
 inline bool al(const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
 
 template <typename TA, int V, int NK, int TAPS>
@@ -508,6 +660,31 @@ int launch_conv(const void* x, long long ldx, const float* w, const float* bias,
   const dim3 grid((groups + 3) / 4, (max_n + chunk - 1) / chunk, entries);
   short_conv_kernel<TA, V, NK, TAPS><<<grid, 128, 0, st>>>(static_cast<const TA*>(x), ldx, w, bias, state, static_cast<TA*>(out), ldo, inv, ldi, sec, taps, C,
                                                             row0, n, ctx, slot, chunk);
+  PG_RET();
+}
+
+// every group 8 * 2^k channels of at most 256, everything on 16-byte boundaries
+inline bool conv_vec_ok(const void* x, long long ldx, const float* w, const float* bias, const float* state, const void* out, long long ldo, int C,
+                        const PgConvSections& sec) {
+  bool ok = al(x, 16) && al(out, 16) && al(w, 16) && al(bias, 16) && al(state, 16) && ldx % 8 == 0 && ldo % 8 == 0 && C % 8 == 0;
+  for (int s = 0; s < sec.count; ++s) {
+    const int l = sec.size[s] / 8;
+    ok = ok && sec.size[s] % 8 == 0 && l > 0 && l <= 32 && (l & (l - 1)) == 0 && sec.total[s] % 8 == 0 && sec.xcol[s] % 8 == 0 && sec.ccol[s] % 8 == 0;
+  }
+  return ok;
+}
+
+template <int TAPS>
+int launch_conv_vec(const void* x, long long ldx, const float* w, const float* bias, float* state, void* out, long long ldo, float* inv, int ldi,
+                    const PgConvSections& sec, int taps, int C, const int* row0, const int* n, const int* ctx, const int* slot, int entries, int max_n,
+                    cudaStream_t st) {
+  int warps = 0;
+  for (int s = 0; s < sec.count; ++s) warps += (sec.total[s] + 255) / 256;
+  int chunk = 64;
+  while (chunk > 8 && (long long)warps * entries * ((max_n + chunk - 1) / chunk) < 16LL * pg::num_sms()) chunk /= 2;
+  const dim3 grid((warps + 3) / 4, (max_n + chunk - 1) / chunk, entries);
+  short_conv_vec_kernel<TAPS><<<grid, 128, 0, st>>>(static_cast<const bf16*>(x), ldx, w, bias, state, static_cast<bf16*>(out), ldo, inv, ldi, sec, taps, C, row0, n,
+                                                     ctx, slot, chunk);
   PG_RET();
 }
 
@@ -550,6 +727,10 @@ extern "C" int pg_short_conv(const void* x, long long ldx, const float* w, const
   if (act_f32) {
     if (taps <= 4) PG_CV(float, 4);
     PG_CV(float, 8);
+  }
+  if (conv_vec_ok(x, ldx, w, bias, state, out, ldo, C, *sec)) {
+    if (taps <= 4) return launch_conv_vec<4>(x, ldx, w, bias, state, out, ldo, inv, ldi, *sec, taps, C, entry_row0, entry_n, entry_ctx, entry_slot, entries, max_n, s);
+    return launch_conv_vec<8>(x, ldx, w, bias, state, out, ldo, inv, ldi, *sec, taps, C, entry_row0, entry_n, entry_ctx, entry_slot, entries, max_n, s);
   }
   if (taps <= 4) PG_CV(bf16, 4);
   PG_CV(bf16, 8);
@@ -631,6 +812,19 @@ extern "C" int pg_group_norm_gate(const float* o, const float* w, int w_n, const
     return gs % v == 0 && ldg % v == 0 && ldo % v == 0 && al(o, 4 * v) && al(w, 4 * v) && al(gate, ab * v) && al(out, ab * v);
   };
   cudaStream_t st = PG_ST(stream);
+  if (fits(4)) {
+    const long long total = (long long)rows * groups;
+    for (int nv = 1; nv <= 8; nv *= 2) {
+      const int lanes = gs / (4 * nv);
+      if (lanes * 4 * nv != gs || lanes > 32 || (lanes & (lanes - 1))) continue;
+      const unsigned blocks = (unsigned)((total + 256 / lanes - 1) / (256 / lanes));
+#define PG_GF(TA, NV) group_norm_gate_flat_kernel<TA, NV><<<blocks, 256, 0, st>>>(o, w, w_n, static_cast<const TA*>(gate), ldg, gate_mode, static_cast<TA*>(out), ldo, D, gs, total, eps, scale)
+      if (act_f32) { if (nv == 1) PG_GF(float, 1); else if (nv == 2) PG_GF(float, 2); else if (nv == 4) PG_GF(float, 4); else PG_GF(float, 8); }
+      else { if (nv == 1) PG_GF(bf16, 1); else if (nv == 2) PG_GF(bf16, 2); else if (nv == 4) PG_GF(bf16, 4); else PG_GF(bf16, 8); }
+#undef PG_GF
+      PG_RET();
+    }
+  }
 #define PG_GN(TA, V) group_norm_gate_kernel<TA, V><<<rows, 256, 0, st>>>(o, w, w_n, static_cast<const TA*>(gate), ldg, gate_mode, static_cast<TA*>(out), ldo, D, groups, eps, scale)
   if (act_f32) {
     if (gs >= 128 && fits(4)) PG_GN(float, 4);

@@ -51,14 +51,32 @@ __device__ __forceinline__ void cut_tiles(const float (&x)[4], const float (&y)[
   cut3(y[0], y[1], a[0][2], a[1][2], a[2][2]);
   cut3(y[2], y[3], a[0][3], a[1][3], a[2][3]);
 }
-// acc += A B for a cut A and a cut B (b0 / b1 = the two halves of the B fragment, per term)
-__device__ __forceinline__ void mma6(float (&acc)[4], const uint32_t (&a)[3][4], const uint32_t* b0, const uint32_t* b1) {
-  mma_bf16_16816(acc, a[0], b0[0], b1[0]);
-  mma_bf16_16816(acc, a[0], b0[1], b1[1]);
-  mma_bf16_16816(acc, a[1], b0[0], b1[0]);
-  mma_bf16_16816(acc, a[1], b0[1], b1[1]);
-  mma_bf16_16816(acc, a[0], b0[2], b1[2]);
-  mma_bf16_16816(acc, a[2], b0[0], b1[0]);
+// acc[i] += A B_i for a cut A and N cut B tiles (b0 / b1 = the halves of the B fragments, [tile][term]); consecutive products go to different
+// accumulators, so that none waits for the one before it
+template <int N>
+__device__ __forceinline__ void mma6(float (&acc)[N][4], const uint32_t (&a)[3][4], const uint32_t (&b0)[N][3], const uint32_t (&b1)[N][3]) {
+  constexpr int TA[6] = {0, 0, 1, 1, 0, 2}, TB[6] = {0, 1, 0, 1, 2, 0};
+#pragma unroll
+  for (int x = 0; x < 6; ++x)
+#pragma unroll
+    for (int i = 0; i < N; ++i) mma_bf16_16816(acc[i], a[TA[x]], b0[i][TB[x]], b1[i][TB[x]]);
+}
+// the same for two tiles with two partial sums each (four chains of three products)
+__device__ __forceinline__ void mma6_pair(float (&acc)[2][4], const uint32_t (&a)[3][4], const uint4 (&f)[3]) {
+  float lo[2][4] = {};
+  const uint32_t b0[2][3] = {{f[0].x, f[1].x, f[2].x}, {f[0].z, f[1].z, f[2].z}}, b1[2][3] = {{f[0].y, f[1].y, f[2].y}, {f[0].w, f[1].w, f[2].w}};
+  constexpr int HA[3] = {0, 1, 0}, HB[3] = {0, 0, 1}, LA[3] = {1, 0, 2}, LB[3] = {1, 2, 0};
+#pragma unroll
+  for (int x = 0; x < 3; ++x) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) mma_bf16_16816(acc[i], a[HA[x]], b0[i][HB[x]], b1[i][HB[x]]);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) mma_bf16_16816(lo[i], a[LA[x]], b0[i][LB[x]], b1[i][LB[x]]);
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) acc[i][c] += lo[i][c];
 }
 
 // S^T fragments <-> the state slot [dim, vdim] (row pitch vdim): thread holds value columns v, v + 8 and key dimensions 8 nb + 2 tq, + 1
@@ -309,16 +327,16 @@ __global__ void __launch_bounds__(128) gated_block_kernel(PgGatedArgs a, int n_m
     for (int kd = 0; kd < DIM / 16; ++kd) {
       uint32_t sa[3][4];
       cut_tiles(S[2 * kd], S[2 * kd + 1], sa);
+      uint32_t bq[C / 16][4];
 #pragma unroll
-      for (int tb = 0; tb < C / 16; ++tb) {
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4(smem_u32(Qb + (tb * 16 + b_row) * LD + kd * 16 + b_col), b0, b1, b2, b3);
+      for (int tb = 0; tb < C / 16; ++tb) ldmatrix_x4(smem_u32(Qb + (tb * 16 + b_row) * LD + kd * 16 + b_col), bq[tb][0], bq[tb][1], bq[tb][2], bq[tb][3]);
 #pragma unroll
-        for (int x = 0; x < 3; ++x) {
-          mma_bf16_16816(o[2 * tb], sa[x], b0, b1);
-          mma_bf16_16816(o[2 * tb + 1], sa[x], b2, b3);
+      for (int x = 0; x < 3; ++x)  // consecutive products go to different accumulators
+#pragma unroll
+        for (int tb = 0; tb < C / 16; ++tb) {
+          mma_bf16_16816(o[2 * tb], sa[x], bq[tb][0], bq[tb][1]);
+          mma_bf16_16816(o[2 * tb + 1], sa[x], bq[tb][2], bq[tb][3]);
         }
-      }
     }
 #pragma unroll
     for (int nb = 0; nb < C / 8; ++nb) {
@@ -330,9 +348,9 @@ __global__ void __launch_bounds__(128) gated_block_kernel(PgGatedArgs a, int n_m
       uint32_t va[4];
       ldmatrix_x4_trans(smem_u32(Vb + (kk * 16 + b_row) * LV + warp * 16 + b_col), va[0], va[1], va[2], va[3]);
 #pragma unroll
-      for (int tb = kk; tb < C / 16; ++tb)
+      for (int x = 0; x < 3; ++x)
 #pragma unroll
-        for (int x = 0; x < 3; ++x) {
+        for (int tb = kk; tb < C / 16; ++tb) {
           uint32_t b0, b1, b2, b3;
           ldmatrix_x4(smem_u32(Ps + (x * C + tb * 16 + b_row) * LP + kk * 16 + b_col), b0, b1, b2, b3);
           mma_bf16_16816(o[2 * tb], va, b0, b1);
@@ -368,14 +386,18 @@ __global__ void __launch_bounds__(128) gated_block_kernel(PgGatedArgs a, int n_m
       cut3(lo_f(va[2]) * u1.x, hi_f(va[2]) * u1.y, wa[0][2], wa[1][2], wa[2][2]);
       cut3(lo_f(va[3]) * u1.x, hi_f(va[3]) * u1.y, wa[0][3], wa[1][3], wa[2][3]);
 #pragma unroll
-      for (int db = 0; db < DIM / 16; ++db) {
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(smem_u32(Kb + (kk * 16 + a_row) * LD + db * 16 + a_col), b0, b1, b2, b3);
+      for (int dp = 0; dp < DIM / 32; ++dp) {
+        uint32_t bk[2][4];
 #pragma unroll
-        for (int x = 0; x < 3; ++x) {
-          mma_bf16_16816(S[2 * db], wa[x], b0, b1);
-          mma_bf16_16816(S[2 * db + 1], wa[x], b2, b3);
-        }
+        for (int hf = 0; hf < 2; ++hf)
+          ldmatrix_x4_trans(smem_u32(Kb + (kk * 16 + a_row) * LD + (2 * dp + hf) * 16 + a_col), bk[hf][0], bk[hf][1], bk[hf][2], bk[hf][3]);
+#pragma unroll
+        for (int x = 0; x < 3; ++x)
+#pragma unroll
+          for (int hf = 0; hf < 2; ++hf) {
+            mma_bf16_16816(S[4 * dp + 2 * hf], wa[x], bk[hf][0], bk[hf][1]);
+            mma_bf16_16816(S[4 * dp + 2 * hf + 1], wa[x], bk[hf][2], bk[hf][3]);
+          }
       }
     }
     if (KIND == 1) {  // every read of the old normaliser was before the barrier above; the next one follows the next barrier
@@ -419,49 +441,82 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(PgDeltaArgs a, float*
   float* Bm = Am + 16 * 17;    // [16][17]
   float* Wm = Bm + 16 * 17;    // [16][17]
   float* bt = Wm + 16 * 17;    // [16]
+  float* iv = bt + 16;         // [2][16] inverse norms of q, k
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int hk = h / (a.H / a.G);
   const bf16* q = static_cast<const bf16*>(a.q) + (long long)hk * dim;
   const bf16* k = static_cast<const bf16*>(a.k) + (long long)hk * dim;
   const float rate = -expf(a.A_log[h]) * LOG2E;
   for (int i = tid; i < 2 * 16 * 17; i += 128) Am[i] = 0.f;  // A and B
-  if (tid < 16) bt[tid] = tid < cn ? 1.0f / (1.0f + expf(-__bfloat162float(static_cast<const bf16*>(a.beta)[(row0 + tid) * a.ldb + h]))) : 0.f;
-  for (int item = tid; item < 2 * DIMP; item += 128) {
-    const int half = item / DIMP, d = item % DIMP;
-    float kv[8], qv[8], lg[8];
+  if (tid < 16) {
+    const bool ok = tid < cn;
+    const float* ivr = a.inv + (row0 + tid) * a.ldi;
+    bt[tid] = ok ? 1.0f / (1.0f + expf(-__bfloat162float(static_cast<const bf16*>(a.beta)[(row0 + tid) * a.ldb + h]))) : 0.f;
+    iv[tid] = ok ? ivr[hk] : 0.f;
+    iv[16 + tid] = ok ? ivr[a.G + hk] : 0.f;
+  }
+  constexpr int ITEMS = (2 * DIMP + 127) / 128;  // (half block, channel) pairs of a thread
+  float lg[ITEMS][8];
+  bf16 kr[ITEMS][8], qr[ITEMS][8];
+  const bf16 zero = __float2bfloat16_rn(0.f);
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int item = tid + it * 128, half = item / DIMP, d = item % DIMP;
+    const bool in = item < 2 * DIMP && d < dim;
+    const int nt = in ? min(8, cn - half * 8) : 0;  // tokens of this half
+    const long long r = row0 + half * 8;
+    const bf16 *kp = k + r * a.ldk + d, *qp = q + r * a.ldq + d;
+    const float* lp = decay + r * a.lda + (long long)h * dim + d;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const int t = half * 8 + i;
-      const bool ok = t < cn && d < dim;
-      kv[i] = ok ? __bfloat162float(k[(row0 + t) * a.ldk + d]) * a.inv[(row0 + t) * a.ldi + a.G + hk] : 0.f;
-      qv[i] = ok ? __bfloat162float(q[(row0 + t) * a.ldq + d]) * a.inv[(row0 + t) * a.ldi + hk] : 0.f;
-      lg[i] = ok ? decay[(row0 + t) * a.lda + (long long)h * dim + d] : 0.f;
+      const bool ok = i < nt;
+      kr[it][i] = ok ? *kp : zero;
+      qr[it][i] = ok ? *qp : zero;
+      lg[it][i] = ok ? *lp : 0.f;
+      kp += a.ldk;
+      qp += a.ldq;
+      lp += a.lda;
     }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int item = tid + it * 128, half = item / DIMP, d = item % DIMP;
+    if (item >= 2 * DIMP) break;
+    const int nt = d < dim ? min(8, cn - half * 8) : 0;
     const float bias = d < dim ? a.dt_bias[(long long)h * dim + d] : 0.f;
     float run = 0.f;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      if (half * 8 + i < cn && d < dim) run = fmaf(rate, softplus(lg[i] + bias), run);
-      lg[i] = run;
+      const float z = lg[it][i] + bias;
+      const float sp = fmaxf(z, 0.f) + log1pf(exp2f(-fabsf(z) * LOG2E));
+      if (i < nt) run = fmaf(rate, sp, run);
+      lg[it][i] = run;
     }
+    const int o = half * 8 * LD + d;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      const int t = half * 8 + i;
-      Lg[t * LD + d] = lg[i];
-      Kn[t * LD + d] = kv[i];
-      Qn[t * LD + d] = qv[i];
-      if (half == 0) Kf[t * LD + d] = kv[i] * exp2f(run - lg[i]);
-      else {
-        const float f = exp2f(lg[i]);
-        Kf[t * LD + d] = kv[i] * f;
-        Qf[i * LD + d] = qv[i] * f;
-      }
+      const float kv = __bfloat162float(kr[it][i]) * iv[16 + half * 8 + i], qv = __bfloat162float(qr[it][i]) * iv[half * 8 + i];
+      Lg[o + i * LD] = lg[it][i];
+      Kn[o + i * LD] = kv;
+      Qn[o + i * LD] = qv;
+      const float f = exp2f(half == 0 ? run - lg[it][i] : lg[it][i]);
+      Kf[o + i * LD] = kv * f;
+      if (half == 1) Qf[i * LD + d] = qv * f;
     }
   }
   __syncthreads();
-  for (int item = tid; item < 16 * dim; item += 128) {  // cumulative over the block, for the sequential part
-    const int t = item / dim, d = item % dim;
-    if (t < cn) decay[(row0 + t) * a.lda + (long long)h * dim + d] = Lg[t * LD + d] + (t >= 8 ? Lg[7 * LD + d] : 0.f);
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {  // cumulative over the block, for the sequential part
+    const int item = tid + it * 128, half = item / DIMP, d = item % DIMP;
+    if (item < 2 * DIMP && d < dim) {
+      const int nt = min(8, cn - half * 8);
+      const float base = half == 1 ? Lg[7 * LD + d] : 0.f;
+      float* lp = decay + (row0 + half * 8) * a.lda + (long long)h * dim + d;
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i < nt) lp[i * a.lda] = lg[it][i] + base;
+    }
   }
   if (warp < 2) {
     // strictly lower pairs of half block `warp`: lane -> (i, j), i > j
@@ -642,19 +697,17 @@ __global__ void __launch_bounds__(128) delta_chain_kernel(PgDeltaArgs a, const u
     const bf16* kg = Tl + cur * 9 * TILE;
     const bf16* qg = kg + 3 * TILE;
     const bf16* ke = qg + 3 * TILE;
-    float xk[2][4] = {}, xq[2][4] = {};
+    float xx[4][4] = {};  // (kg S)^T of the two halves of the block, then (qg S)^T
 #pragma unroll
     for (int kd = 0; kd < DIM / 16; ++kd) {
-      uint32_t sa[3][4], b0[2][3], b1[2][3];
+      uint32_t sa[3][4], b0[4][3], b1[4][3];
       cut_tiles(S[2 * kd], S[2 * kd + 1], sa);
 #pragma unroll
-      for (int x = 0; x < 3; ++x) ldmatrix_x4(smem_u32(kg + x * TILE + b_row * LD + kd * 16 + b_col), b0[0][x], b1[0][x], b0[1][x], b1[1][x]);
-      mma6(xk[0], sa, b0[0], b1[0]);
-      mma6(xk[1], sa, b0[1], b1[1]);
-#pragma unroll
-      for (int x = 0; x < 3; ++x) ldmatrix_x4(smem_u32(qg + x * TILE + b_row * LD + kd * 16 + b_col), b0[0][x], b1[0][x], b0[1][x], b1[1][x]);
-      mma6(xq[0], sa, b0[0], b1[0]);
-      mma6(xq[1], sa, b0[1], b1[1]);
+      for (int x = 0; x < 3; ++x) {
+        ldmatrix_x4(smem_u32(kg + x * TILE + b_row * LD + kd * 16 + b_col), b0[0][x], b1[0][x], b0[1][x], b1[1][x]);
+        ldmatrix_x4(smem_u32(qg + x * TILE + b_row * LD + kd * 16 + b_col), b0[2][x], b1[2][x], b0[3][x], b1[3][x]);
+      }
+      mma6<4>(xx, sa, b0, b1);
     }
     // R^T = V^T - (kg S)^T, U^T = R^T W^T
     uint32_t va[4], ra[3][4];
@@ -662,25 +715,18 @@ __global__ void __launch_bounds__(128) delta_chain_kernel(PgDeltaArgs a, const u
     float u[2][4];
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb) {
-      u[nb][0] = lo_f(va[2 * nb]) - xk[nb][0]; u[nb][1] = hi_f(va[2 * nb]) - xk[nb][1];
-      u[nb][2] = lo_f(va[2 * nb + 1]) - xk[nb][2]; u[nb][3] = hi_f(va[2 * nb + 1]) - xk[nb][3];
+      u[nb][0] = lo_f(va[2 * nb]) - xx[nb][0]; u[nb][1] = hi_f(va[2 * nb]) - xx[nb][1];
+      u[nb][2] = lo_f(va[2 * nb + 1]) - xx[nb][2]; u[nb][3] = hi_f(va[2 * nb + 1]) - xx[nb][3];
     }
     cut_tiles(u[0], u[1], ra);
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb) u[nb][0] = u[nb][1] = u[nb][2] = u[nb][3] = 0.f;
-    {
-      const uint32_t b00[3] = {fw[0].x, fw[1].x, fw[2].x}, b01[3] = {fw[0].y, fw[1].y, fw[2].y};
-      const uint32_t b10[3] = {fw[0].z, fw[1].z, fw[2].z}, b11[3] = {fw[0].w, fw[1].w, fw[2].w};
-      mma6(u[0], ra, b00, b01);
-      mma6(u[1], ra, b10, b11);
-    }
+    mma6_pair(u, ra, fw);
     cut_tiles(u[0], u[1], ra);
-    {
-      const uint32_t b00[3] = {fb[0].x, fb[1].x, fb[2].x}, b01[3] = {fb[0].y, fb[1].y, fb[2].y};
-      const uint32_t b10[3] = {fb[0].z, fb[1].z, fb[2].z}, b11[3] = {fb[0].w, fb[1].w, fb[2].w};
-      mma6(xq[0], ra, b00, b01);
-      mma6(xq[1], ra, b10, b11);
-    }
+    float y[2][4];
+#pragma unroll
+    for (int nb = 0; nb < 2; ++nb) { y[nb][0] = xx[2 + nb][0]; y[nb][1] = xx[2 + nb][1]; y[nb][2] = xx[2 + nb][2]; y[nb][3] = xx[2 + nb][3]; }
+    mma6_pair(y, ra, fb);
     if (more) {
       frag += frag_step;
 #pragma unroll
@@ -691,21 +737,26 @@ __global__ void __launch_bounds__(128) delta_chain_kernel(PgDeltaArgs a, const u
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int t = t0 + nb * 8 + 2 * tq + (i & 1), c = vcol + (i >> 1) * 8;
-        if (t < n && c < vdim) a.out[(row0 + t) * ((long long)H * vdim) + (long long)h * vdim + c] = xq[nb][i];
+        if (t < n && c < vdim) a.out[(row0 + t) * ((long long)H * vdim) + (long long)h * vdim + c] = y[nb][i];
       }
 #pragma unroll
-    for (int db = 0; db < DIM / 16; ++db) {
+    for (int dp = 0; dp < DIM / 32; ++dp) {
+      uint32_t b0[4][3], b1[4][3];
 #pragma unroll
-      for (int nb = 0; nb < 2; ++nb) {
-        const float2 g = *reinterpret_cast<const float2*>(Ge + cur * DIM + db * 16 + nb * 8 + 2 * tq);
-        float(&s)[4] = S[2 * db + nb];
-        s[0] *= g.x; s[1] *= g.y; s[2] *= g.x; s[3] *= g.y;
+      for (int x = 0; x < 3; ++x)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf)
+          ldmatrix_x4_trans(smem_u32(ke + x * TILE + a_row * LD + (2 * dp + hf) * 16 + a_col), b0[2 * hf][x], b1[2 * hf][x], b0[2 * hf + 1][x], b1[2 * hf + 1][x]);
+      float acc[4][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 g = *reinterpret_cast<const float2*>(Ge + cur * DIM + dp * 32 + i * 8 + 2 * tq);
+        const float(&st)[4] = S[4 * dp + i];
+        acc[i][0] = st[0] * g.x; acc[i][1] = st[1] * g.y; acc[i][2] = st[2] * g.x; acc[i][3] = st[3] * g.y;
       }
-      uint32_t b0[2][3], b1[2][3];
+      mma6<4>(acc, ra, b0, b1);
 #pragma unroll
-      for (int x = 0; x < 3; ++x) ldmatrix_x4_trans(smem_u32(ke + x * TILE + a_row * LD + db * 16 + a_col), b0[0][x], b1[0][x], b0[1][x], b1[1][x]);
-      mma6(S[2 * db], ra, b0[0], b1[0]);
-      mma6(S[2 * db + 1], ra, b0[1], b1[1]);
+      for (int i = 0; i < 4; ++i) { S[4 * dp + i][0] = acc[i][0]; S[4 * dp + i][1] = acc[i][1]; S[4 * dp + i][2] = acc[i][2]; S[4 * dp + i][3] = acc[i][3]; }
     }
   }
   store_state<DIM>(S, stp, dim, vdim, vcol, tq);
@@ -734,7 +785,7 @@ int launch_gated(const PgGatedArgs& a, int n_min, cudaStream_t st) {
 template <int DIM>
 int launch_delta(const PgDeltaArgs& a, float* decay, uint4* scratch, int max_n, int n_min, cudaStream_t st) {
   constexpr int DP = (DIM + 31) / 32 * 32;
-  const size_t s1 = (size_t)(72 * (DP + 4) + 3 * 16 * 17 + 16) * sizeof(float);
+  const size_t s1 = (size_t)(72 * (DP + 4) + 3 * 16 * 17 + 48) * sizeof(float);
   auto k1 = delta_blocks_kernel<DP>;
   int rc = set_smem(k1, s1);
   if (rc != PG_OK) return rc;
