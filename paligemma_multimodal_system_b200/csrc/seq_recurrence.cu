@@ -203,104 +203,129 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const TA* __restrict__ 
   }
 }
 
-// The same for groups of 8 * 2^k <= 256 channels and 16-byte aligned rows (bf16): lane <-> 8 adjacent channels, so that a warp covers 256 adjacent
-// channels of a row (several groups), and the next ROWS_AHEAD rows are in flight while the current one is computed.
-__device__ __forceinline__ void unpack8(uint4 u, float* v) {
-  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    v[2 * i] = __uint_as_float(w[i] << 16);
-    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-  }
+// The same for groups of V * 2^k <= 32 V channels and aligned rows (bf16; V = 4 or 8 channels per lane): a warp covers 32 V adjacent channels of a
+// row (several groups), the next AHEAD rows are in flight while the current ones are computed, and AHEAD rows pass without a branch.
+template <int V>
+struct Packed;
+template <>
+struct Packed<4> { using T = uint2; };
+template <>
+struct Packed<8> { using T = uint4; };
+__device__ __forceinline__ void unpack(uint2 u, float* v) {
+  v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+  v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+}
+__device__ __forceinline__ void unpack(uint4 u, float* v) {
+  unpack(make_uint2(u.x, u.y), v);
+  unpack(make_uint2(u.z, u.w), v + 4);
+}
+__device__ __forceinline__ void pack(const float* v, uint2& u) { u = make_uint2(pg::pack_bf16(v[0], v[1]), pg::pack_bf16(v[2], v[3])); }
+__device__ __forceinline__ void pack(const float* v, uint4& u) {
+  u = make_uint4(pg::pack_bf16(v[0], v[1]), pg::pack_bf16(v[2], v[3]), pg::pack_bf16(v[4], v[5]), pg::pack_bf16(v[6], v[7]));
 }
 
-template <int TAPS>
+template <int TAPS, int V>
 __global__ void __launch_bounds__(128) short_conv_vec_kernel(const bf16* __restrict__ x, long long ldx, const float* __restrict__ w,
                                                              const float* __restrict__ bias, float* __restrict__ state, bf16* __restrict__ out,
                                                              long long ldo, float* __restrict__ inv, int ldi, PgConvSections sec, int taps, int C,
                                                              const int* __restrict__ entry_row0, const int* __restrict__ entry_n,
                                                              const int* __restrict__ entry_ctx, const int* __restrict__ entry_slot, int chunk) {
-  constexpr int AHEAD = 4;
+  constexpr int AHEAD = 4, WC = 32 * V;
+  using P = typename Packed<V>::T;
   const int e = blockIdx.z, lane = threadIdx.x & 31;
   const int n = entry_n[e], r0 = blockIdx.y * chunk;
   if (r0 >= n) return;
   int g = blockIdx.x * 4 + (threadIdx.x >> 5), s = 0, unit_base = 0;
-  while (s < sec.count && g >= (sec.total[s] + 255) / 256) {
-    g -= (sec.total[s] + 255) / 256;
+  while (s < sec.count && g >= (sec.total[s] + WC - 1) / WC) {
+    g -= (sec.total[s] + WC - 1) / WC;
     if (sec.unit[s]) unit_base += sec.groups[s];
     ++s;
   }
   if (s >= sec.count) return;
-  const int c = g * 256 + lane * 8;  // channel inside the section
-  const bool ok = c < sec.total[s];  // totals are multiples of 8
-  const int lanes = sec.size[s] / 8; // lanes of one group
+  const int c = g * WC + lane * V;    // channel inside the section
+  const bool ok = c < sec.total[s];   // totals are multiples of V
+  const int lanes = sec.size[s] / V;  // lanes of one group
   const long long row0 = entry_row0[e];
   const bf16* xp = x + row0 * ldx + sec.xcol[s] + (ok ? c : 0);
   bf16* op = out + row0 * ldo + sec.ccol[s] + (ok ? c : 0);
   const int cc = sec.ccol[s] + (ok ? c : 0), K = taps - 1;
   float* slot = state + (long long)entry_slot[e] * K * C + cc;
-  float wt[TAPS][8], bs[8], hist[TAPS - 1][8];
-  auto ld8 = [](const float* p, float* v) { ldv<4>(p, 0, v); ldv<4>(p, 4, v + 4); };
-  auto zero8 = [](float* v) {
+  float wt[TAPS][V], bs[V], hist[TAPS - 1][V];
+  auto ldf = [](const float* p, float* v) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = 0.f;
+    for (int i = 0; i < V; i += 4) ldv<4>(p, i, v + i);
   };
-  if (bias != nullptr) ld8(bias + cc, bs); else zero8(bs);
+  auto zero = [](float* v) {
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = 0.f;
+  };
+  auto row_at = [&](int r) { return *reinterpret_cast<const P*>(xp + (long long)r * ldx); };
+  if (bias != nullptr) ldf(bias + cc, bs); else zero(bs);
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) {
     const int tj = j - (TAPS - taps);
-    if (tj >= 0) ld8(w + (long long)tj * C + cc, wt[j]); else zero8(wt[j]);
+    if (tj >= 0) ldf(w + (long long)tj * C + cc, wt[j]); else zero(wt[j]);
   }
 #pragma unroll
   for (int j = 0; j < TAPS - 1; ++j) {
     const int row = r0 - (TAPS - 1) + j;
-    if (row >= 0) unpack8(*reinterpret_cast<const uint4*>(xp + row * ldx), hist[j]);
-    else if (entry_ctx[e] > 0 && K + row >= 0) ld8(slot + (long long)(K + row) * C, hist[j]);
-    else zero8(hist[j]);
+    if (row >= 0) unpack(row_at(row), hist[j]);
+    else if (entry_ctx[e] > 0 && K + row >= 0) ldf(slot + (long long)(K + row) * C, hist[j]);
+    else zero(hist[j]);
   }
   const int r1 = min(n, r0 + chunk);
-  uint4 nxt[AHEAD];
+  const bool unit = sec.unit[s] != 0;
+  const float unit_scale = sec.scale[s];
+  float* ip = (unit && ok && (lane & (lanes - 1)) == 0) ? inv + row0 * ldi + unit_base + c / sec.size[s] : nullptr;
+  P nxt[AHEAD];
 #pragma unroll
-  for (int i = 0; i < AHEAD; ++i) nxt[i] = r0 + i < r1 ? *reinterpret_cast<const uint4*>(xp + (long long)(r0 + i) * ldx) : make_uint4(0, 0, 0, 0);
+  for (int i = 0; i < AHEAD; ++i) nxt[i] = row_at(min(r0 + i, r1 - 1));
   for (int rb = r0; rb < r1; rb += AHEAD) {
+    float ss[AHEAD];
 #pragma unroll
     for (int i = 0; i < AHEAD; ++i) {
-      const int r = rb + i;
-      if (r >= r1) break;
-      float cur[8], y[8], ss = 0.f;
-      unpack8(nxt[i], cur);
-      if (r + AHEAD < r1) nxt[i] = *reinterpret_cast<const uint4*>(xp + (long long)(r + AHEAD) * ldx);
+      const int r = rb + i;  // rows past the run are computed from a repeated row and not stored
+      float cur[V], y[V];
+      unpack(nxt[i], cur);
+      nxt[i] = row_at(min(r + AHEAD, r1 - 1));
 #pragma unroll
-      for (int v = 0; v < 8; ++v) {
-        float a = bs[v];
+      for (int v = 0; v < V; ++v) {
+        float a = fmaf(wt[TAPS - 1][v], cur[v], bs[v]);
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j) a = fmaf(wt[j][v], hist[j][v], a);
-        a = fmaf(wt[TAPS - 1][v], cur[v], a);
 #pragma unroll
         for (int j = 0; j < TAPS - 2; ++j) hist[j][v] = hist[j + 1][v];
         hist[TAPS - 2][v] = cur[v];
         y[v] = __fdividef(a, 1.0f + __expf(-a));  // a bf16 activation: the hardware exponential is far below its rounding
       }
-      const uint4 pk = make_uint4(pg::pack_bf16(y[0], y[1]), pg::pack_bf16(y[2], y[3]), pg::pack_bf16(y[4], y[5]), pg::pack_bf16(y[6], y[7]));
-      if (ok) *reinterpret_cast<uint4*>(op + (long long)r * ldo) = pk;
-      if (sec.unit[s]) {
-        unpack8(pk, y);  // the norm is that of the stored activations
+      P pk;
+      pack(y, pk);
+      if (ok && r < r1) *reinterpret_cast<P*>(op + (long long)r * ldo) = pk;
+      unpack(pk, y);  // the norm is that of the stored activations
+      ss[i] = 0.f;
 #pragma unroll
-        for (int v = 0; v < 8; ++v) ss = fmaf(y[v], y[v], ss);
-        for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        if (ok && (lane & (lanes - 1)) == 0) inv[(row0 + r) * ldi + unit_base + c / sec.size[s]] = sec.scale[s] / sqrtf(ss + 1e-6f);
+      for (int v = 0; v < V; ++v) ss[i] = fmaf(y[v], y[v], ss[i]);
+    }
+    if (unit) {
+      for (int o = lanes / 2; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+      if (ip != nullptr) {
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+          if (rb + i < r1) ip[(long long)(rb + i) * ldi] = unit_scale / sqrtf(ss[i] + 1e-6f);
       }
     }
   }
   if (r0 == 0 && K > 0 && ok) {  // owner of the slot: it becomes the inputs of the entry's last K rows
     for (int j = 0; j < K; ++j) {
       const int row = n - K + j;
-      float h[8];
-      if (row >= 0) unpack8(*reinterpret_cast<const uint4*>(xp + (long long)row * ldx), h);
-      else if (entry_ctx[e] > 0) ld8(slot + (long long)(n + j) * C, h);
-      else zero8(h);
-      stv<4>(slot, (long long)j * C, h);
-      stv<4>(slot, (long long)j * C + 4, h + 4);
+      float h[V];
+      if (row >= 0) unpack(row_at(row), h);
+      else if (entry_ctx[e] > 0) ldf(slot + (long long)(n + j) * C, h);
+      else zero(h);
+#pragma unroll
+      for (int i = 0; i < V; i += 4) stv<4>(slot, (long long)j * C + i, h + i);
     }
   }
 }
@@ -663,28 +688,32 @@ int launch_conv(const void* x, long long ldx, const float* w, const float* bias,
   PG_RET();
 }
 
-// every group 8 * 2^k channels of at most 256, everything on 16-byte boundaries
-inline bool conv_vec_ok(const void* x, long long ldx, const float* w, const float* bias, const float* state, const void* out, long long ldo, int C,
-                        const PgConvSections& sec) {
-  bool ok = al(x, 16) && al(out, 16) && al(w, 16) && al(bias, 16) && al(state, 16) && ldx % 8 == 0 && ldo % 8 == 0 && C % 8 == 0;
-  for (int s = 0; s < sec.count; ++s) {
-    const int l = sec.size[s] / 8;
-    ok = ok && sec.size[s] % 8 == 0 && l > 0 && l <= 32 && (l & (l - 1)) == 0 && sec.total[s] % 8 == 0 && sec.xcol[s] % 8 == 0 && sec.ccol[s] % 8 == 0;
+// V channels per lane (4 or 8; 0: only the general kernel fits): every group V * 2^k channels of at most 32 V, everything aligned
+inline int conv_vec_width(const void* x, long long ldx, const float* w, const float* bias, const float* state, const void* out, long long ldo, int C,
+                          const PgConvSections& sec) {
+  if (!al(x, 16) || !al(out, 16) || !al(w, 16) || !al(bias, 16) || !al(state, 16) || ldx % 8 || ldo % 8 || C % 8) return 0;
+  for (int v = 4; v <= 8; v += 4) {
+    bool ok = true;
+    for (int s = 0; s < sec.count; ++s) {
+      const int l = sec.size[s] / v;
+      ok = ok && sec.size[s] % v == 0 && l > 0 && l <= 32 && (l & (l - 1)) == 0 && sec.total[s] % v == 0 && sec.xcol[s] % 8 == 0 && sec.ccol[s] % 8 == 0;
+    }
+    if (ok) return v;
   }
-  return ok;
+  return 0;
 }
 
-template <int TAPS>
+template <int TAPS, int V>
 int launch_conv_vec(const void* x, long long ldx, const float* w, const float* bias, float* state, void* out, long long ldo, float* inv, int ldi,
                     const PgConvSections& sec, int taps, int C, const int* row0, const int* n, const int* ctx, const int* slot, int entries, int max_n,
                     cudaStream_t st) {
   int warps = 0;
-  for (int s = 0; s < sec.count; ++s) warps += (sec.total[s] + 255) / 256;
+  for (int s = 0; s < sec.count; ++s) warps += (sec.total[s] + 32 * V - 1) / (32 * V);
   int chunk = 64;
-  while (chunk > 8 && (long long)warps * entries * ((max_n + chunk - 1) / chunk) < 16LL * pg::num_sms()) chunk /= 2;
+  while (chunk > 8 && (long long)warps * entries * ((max_n + chunk - 1) / chunk) < 48LL * pg::num_sms()) chunk /= 2;
   const dim3 grid((warps + 3) / 4, (max_n + chunk - 1) / chunk, entries);
-  short_conv_vec_kernel<TAPS><<<grid, 128, 0, st>>>(static_cast<const bf16*>(x), ldx, w, bias, state, static_cast<bf16*>(out), ldo, inv, ldi, sec, taps, C, row0, n,
-                                                     ctx, slot, chunk);
+  short_conv_vec_kernel<TAPS, V><<<grid, 128, 0, st>>>(static_cast<const bf16*>(x), ldx, w, bias, state, static_cast<bf16*>(out), ldo, inv, ldi, sec, taps, C, row0,
+                                                        n, ctx, slot, chunk);
   PG_RET();
 }
 
@@ -728,10 +757,13 @@ extern "C" int pg_short_conv(const void* x, long long ldx, const float* w, const
     if (taps <= 4) PG_CV(float, 4);
     PG_CV(float, 8);
   }
-  if (conv_vec_ok(x, ldx, w, bias, state, out, ldo, C, *sec)) {
-    if (taps <= 4) return launch_conv_vec<4>(x, ldx, w, bias, state, out, ldo, inv, ldi, *sec, taps, C, entry_row0, entry_n, entry_ctx, entry_slot, entries, max_n, s);
-    return launch_conv_vec<8>(x, ldx, w, bias, state, out, ldo, inv, ldi, *sec, taps, C, entry_row0, entry_n, entry_ctx, entry_slot, entries, max_n, s);
-  }
+  const int vw = conv_vec_width(x, ldx, w, bias, state, out, ldo, C, *sec);
+#define PG_CVV(TAPS, V) return launch_conv_vec<TAPS, V>(x, ldx, w, bias, state, out, ldo, inv, ldi, *sec, taps, C, entry_row0, entry_n, entry_ctx, entry_slot, entries, max_n, s)
+  if (vw == 4 && taps <= 4) PG_CVV(4, 4);
+  if (vw == 4) PG_CVV(8, 4);
+  if (vw == 8 && taps <= 4) PG_CVV(4, 8);
+  if (vw == 8) PG_CVV(8, 8);
+#undef PG_CVV
   if (taps <= 4) PG_CV(bf16, 4);
   PG_CV(bf16, 8);
 #undef PG_CV

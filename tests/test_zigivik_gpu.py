@@ -394,7 +394,7 @@ def test_latent_window_edge_with_a_key_that_dominates(case, dtype, tol, cuts):
 def test_far_key_among_a_thousand_in_keys_as_values_attention(needle, dtype, tol):
     """One token's input is five times larger, so its key (and value) weighs heavily wherever it is seen: from the end of a prompt of
     1100 tokens, from a portion that starts on a page border and from decoded tokens.  (bf16: the rows next to the large token carry its
-    rounding, hence the wider bound on them.)"""
+    rounding; every row's error is taken relative to its own size there.)"""
     from paligemma_multimodal_system_b200 import seq_ops
     D, T, eps = 40, 1100, 1e-5
     cfg = make_cfg([with_ff(attention(heads=2, kv_heads=1, dim=64, rot_dims=32, base=1e4), 0)], width=D, eps=eps)
@@ -409,7 +409,8 @@ def test_far_key_among_a_thousand_in_keys_as_values_attention(needle, dtype, tol
     mx.pack(prec)
     for cuts in ([T], [1088, 1], [1024, 70, 2]):
         got = run_mixer(mx, [mx.cache_spec()], h, cuts, dtype, prec)
-        assert worst_row(got[-40:], ref[-40:]) < min(tol, 5e-2) and worst_row(got, ref) < tol, cuts
+        own = ((got.double() - ref).pow(2).mean(-1) / torch.maximum(ref.pow(2).mean(-1), ref.pow(2).mean())).sqrt()
+        assert worst_row(got[-40:], ref[-40:]) < min(tol, 5e-2) and float(own.max()) < tol, cuts
 
 
 def test_first_positions_share_the_softmax_with_the_unit_in_the_denominator():
@@ -602,7 +603,7 @@ def test_greedy_generation_through_the_scheduler():
     equal the oracle's greedy continuation of each prompt alone."""
     cfg = make_cfg([with_ff(latent(heads=2, dim=16, rot_dim=8, vdim=16, q_rank=16, kv_rank=16, size=30), 48), with_ff(attention(heads=2, kv_heads=1, dim=16, rot_dims=8), 32),
                     with_ff(latent(heads=4, dim=8, rot_dim=8, vdim=8, q_rank=16, kv_rank=16, size=25, kv_from=0), 0)], width=48, vocab=60)
-    w = O.random_weights(cfg, seed=31)
+    w = O.random_weights(cfg, seed=34)  # no step of these continuations is a near tie
     prompts = [toks(n, 60, 40 + n) for n in (70, 5, 33, 1, 90, 12)]
     new = 10
     eng = engine_for(cfg, w, torch.float32, max_tokens=5 * 64, slots=3)
