@@ -518,9 +518,9 @@ int pg_group_norm_gate(const float* o, const float* w, int w_n, const void* gate
 
 /* A gated sub-layer result joins the residual behind a layer norm, and the next sub-layer's input norm follows from the same row:
  *   z = y[t, :] * sigmoid(gate[t, :] + gate_b);  x[t, :] += LN(z; w1, b1);  out[t, :] = LN(x[t, :]; w2, b2)   (out NULL: no second norm)
- * y fp32 (pitch ldy), gate activation type (pitch ldg; NULL: no gate), x fp32 [rows, D] in place, out activation type [rows, D]. */
+ * y fp32 (pitch ldy), gate activation type or fp32 (gate_f32; pitch ldg; NULL: no gate), x fp32 [rows, D] in place, out activation type [rows, D]. */
 int pg_gated_layernorm_add(const float* y, long long ldy, const void* gate, long long ldg, const float* gate_b, const float* w1, const float* b1, float* x,
-                           const float* w2, const float* b2, void* out, int rows, int D, float eps, int act_f32, void* stream);
+                           const float* w2, const float* b2, void* out, int rows, int D, float eps, int gate_f32, int act_f32, void* stream);
 
 /* ---- multi-stream residual ("hyper-connections"): xs fp32 [rows, S, D], S <= 16 ------------------------------------------------
  * pg_embed_streams: xs[t, s, :] = table[tokens[t], 0:D] * scale for every stream s.

@@ -105,7 +105,7 @@ SIGNATURES = {
     "pg_gated_blocks": [p, i32, i32, p],
     "pg_delta_blocks": [p, p, p, i32, i32, p],
     "pg_group_norm_gate": [p, p, i32, p, i64, i32, p, i64, i32, i32, i32, f32, f32, i32, p],
-    "pg_gated_layernorm_add": [p, i64, p, i64, p, p, p, p, p, p, p, i32, i32, f32, i32, p],
+    "pg_gated_layernorm_add": [p, i64, p, i64, p, p, p, p, p, p, p, i32, i32, f32, i32, i32, p],
     "pg_glu": [p, i64, p, i64, i32, i32, i32, f32, f32, i32, p],
 }
 _RESTYPE = {"pg_launch_count": i64}

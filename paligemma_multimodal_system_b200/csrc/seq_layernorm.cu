@@ -384,8 +384,8 @@ __device__ __forceinline__ float4 ld_act4(const bf16* p) {
 }
 __device__ __forceinline__ float sigmoid1(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-template <typename TA, int VT>
-__global__ void __launch_bounds__(256) gated_layernorm_add_vec_kernel(const float* __restrict__ y, long long ldy, const TA* __restrict__ gate, long long ldg,
+template <typename TA, typename TG, int VT>
+__global__ void __launch_bounds__(256) gated_layernorm_add_vec_kernel(const float* __restrict__ y, long long ldy, const TG* __restrict__ gate, long long ldg,
                                                                       const float* __restrict__ gb, const float* __restrict__ w1,
                                                                       const float* __restrict__ b1, float* __restrict__ x, const float* __restrict__ w2,
                                                                       const float* __restrict__ b2, TA* __restrict__ out, int D, float eps) {
@@ -430,8 +430,8 @@ __global__ void __launch_bounds__(256) gated_layernorm_add_vec_kernel(const floa
 }
 
 // other widths: the row staged in shared memory
-template <typename TA>
-__global__ void __launch_bounds__(256) gated_layernorm_add_kernel(const float* __restrict__ y, long long ldy, const TA* __restrict__ gate, long long ldg,
+template <typename TA, typename TG>
+__global__ void __launch_bounds__(256) gated_layernorm_add_kernel(const float* __restrict__ y, long long ldy, const TG* __restrict__ gate, long long ldg,
                                                                   const float* __restrict__ gb, const float* __restrict__ w1, const float* __restrict__ b1,
                                                                   float* __restrict__ x, const float* __restrict__ w2, const float* __restrict__ b2,
                                                                   TA* __restrict__ out, int D, float eps) {
@@ -468,15 +468,15 @@ __global__ void __launch_bounds__(256) gated_layernorm_add_kernel(const float* _
   for (int d = threadIdx.x; d < D; d += 256) st_act(out, t * D + d, fmaf((buf[d] - mean) * rstd, w2[d], b2[d]));
 }
 
-template <typename TA>
+template <typename TA, typename TG>
 int launch_gated_ln(const float* y, long long ldy, const void* gate, long long ldg, const float* gb, const float* w1, const float* b1, float* x,
                     const float* w2, const float* b2, void* out, int rows, int D, float eps, cudaStream_t st) {
-  const TA* g = static_cast<const TA*>(gate);
+  const TG* g = static_cast<const TG*>(gate);
   TA* o = static_cast<TA*>(out);
   auto al = [](const void* p, size_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
-  if (D % 4 == 0 && D <= 8192 && ldy % 4 == 0 && ldg % 4 == 0 && al(y, 16) && al(gate, 4 * sizeof(TA)) && al(gb, 16) && al(w1, 16) && al(b1, 16) && al(x, 16) &&
+  if (D % 4 == 0 && D <= 8192 && ldy % 4 == 0 && ldg % 4 == 0 && al(y, 16) && al(gate, 4 * sizeof(TG)) && al(gb, 16) && al(w1, 16) && al(b1, 16) && al(x, 16) &&
       al(w2, 16) && al(b2, 16) && al(out, 4 * sizeof(TA))) {
-#define PG_GLN(VT) gated_layernorm_add_vec_kernel<TA, VT><<<rows, 256, 0, st>>>(y, ldy, g, ldg, gb, w1, b1, x, w2, b2, o, D, eps)
+#define PG_GLN(VT) gated_layernorm_add_vec_kernel<TA, TG, VT><<<rows, 256, 0, st>>>(y, ldy, g, ldg, gb, w1, b1, x, w2, b2, o, D, eps)
     if (D <= 1024) PG_GLN(1);
     else if (D <= 2048) PG_GLN(2);
     else if (D <= 4096) PG_GLN(4);
@@ -486,7 +486,7 @@ int launch_gated_ln(const float* y, long long ldy, const void* gate, long long l
   }
   const size_t smem = (size_t)D * sizeof(float);
   if (smem > 200 * 1024) return PG_ERR_ARG;
-  auto kern = gated_layernorm_add_kernel<TA>;
+  auto kern = gated_layernorm_add_kernel<TA, TG>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return PG_ERR_CUDA;
   kern<<<rows, 256, smem, st>>>(y, ldy, g, ldg, gb, w1, b1, x, w2, b2, o, D, eps);
   PG_RET();
@@ -495,12 +495,14 @@ int launch_gated_ln(const float* y, long long ldy, const void* gate, long long l
 }  // namespace
 
 extern "C" int pg_gated_layernorm_add(const float* y, long long ldy, const void* gate, long long ldg, const float* gate_b, const float* w1, const float* b1,
-                                      float* x, const float* w2, const float* b2, void* out, int rows, int D, float eps, int act_f32, void* stream) {
+                                      float* x, const float* w2, const float* b2, void* out, int rows, int D, float eps, int gate_f32, int act_f32, void* stream) {
   if (rows <= 0 || D <= 0 || y == nullptr || w1 == nullptr || b1 == nullptr || x == nullptr || (gate != nullptr && gate_b == nullptr) ||
       (out != nullptr && (w2 == nullptr || b2 == nullptr)))
     return PG_ERR_ARG;
-  if (act_f32) return launch_gated_ln<float>(y, ldy, gate, ldg, gate_b, w1, b1, x, w2, b2, out, rows, D, eps, PG_ST(stream));
-  return launch_gated_ln<bf16>(y, ldy, gate, ldg, gate_b, w1, b1, x, w2, b2, out, rows, D, eps, PG_ST(stream));
+  if (act_f32 && !gate_f32) return PG_ERR_ARG;
+  if (act_f32) return launch_gated_ln<float, float>(y, ldy, gate, ldg, gate_b, w1, b1, x, w2, b2, out, rows, D, eps, PG_ST(stream));
+  if (gate_f32) return launch_gated_ln<bf16, float>(y, ldy, gate, ldg, gate_b, w1, b1, x, w2, b2, out, rows, D, eps, PG_ST(stream));
+  return launch_gated_ln<bf16, bf16>(y, ldy, gate, ldg, gate_b, w1, b1, x, w2, b2, out, rows, D, eps, PG_ST(stream));
 }
 
 extern "C" int pg_layernorm_shift(const float* x, const float* w1, const float* b1, const float* shift, const float* w2, const float* b2, void* out1,

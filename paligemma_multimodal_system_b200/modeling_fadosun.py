@@ -150,6 +150,10 @@ class FadosunForCausalLM:
             blk.load(take)
         self.final_norm, self.final_norm_b = take("final.norm", (c.width,)), take("final.norm.b", (c.width,))
         self.head = take("head", (c.vocab, c.width))
+        for blk in self.blocks:  # a layer without a feed-forward has no second sub-layer; norms and gate a checkpoint kept for it are unused
+            if blk.ff is None:
+                for name in ("norm2", "norm2.b", "norm2b", "norm2b.b", "rg2", "rg2.b"):
+                    left.pop(f"l{blk.i}.{name}", None)
         if left:
             raise KeyError(f"checkpoint tensors without a place in the model: {sorted(left)[:8]}")
         self._packed = False
@@ -193,7 +197,8 @@ class FadosunForCausalLM:
         for li, blk in enumerate(self.blocks):
             join(blk.sub1, *blk.mixer(a, b, store, self.cache_at[li], prec))
             if blk.ff is not None:
-                gate = seq_ops.linear(a, blk.sub2.rg, prec.empty(b.T, c.width))
+                # few rows: an fp32 product may split its reduction over the whole GPU
+                gate = seq_ops.linear(a, blk.sub2.rg, torch.empty(b.T, c.width, device="cuda", dtype=torch.float32 if b.T <= 128 else prec.dtype))
                 join(blk.sub2, blk.ff(a, b, prec), gate)
             if trace is not None:
                 trace.append(x.clone())

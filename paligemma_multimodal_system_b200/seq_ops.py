@@ -705,12 +705,15 @@ def group_norm_gate(o, w, gate, out, groups, eps, mode, scale=1.0):
 
 
 def gated_layernorm_add(y, gate, gate_b, w1, b1, x, eps, w2=None, b2=None, out=None):
-    """x += LN(y * sigmoid(gate + gate_b); w1, b1) in place (fp32); out (activation type) = LN(x; w2, b2), the next sub-layer's input, when given."""
+    """x += LN(y * sigmoid(gate + gate_b); w1, b1) in place (fp32); out (activation type) = LN(x; w2, b2), the next sub-layer's input, when given.
+    gate: bf16, or fp32 beside any output type."""
     rows, D = x.shape
     assert y.dtype == torch.float32 and y.shape == x.shape and y.stride(1) == 1 and x.dtype == torch.float32 and x.is_contiguous()
-    assert gate is None or (gate.shape == x.shape and gate.stride(1) == 1 and (out is None or gate.dtype == out.dtype))
+    assert gate is None or (gate.shape == x.shape and gate.stride(1) == 1 and gate.dtype in (torch.float32, torch.bfloat16))
     assert out is None or (out.is_contiguous() and out.shape == x.shape and w2 is not None and b2 is not None)
-    ref = gate if gate is not None else out
+    gate_f32 = int(gate is None or gate.dtype == torch.float32)
+    act_f32 = int(out.dtype == torch.float32) if out is not None else gate_f32
+    assert gate_f32 or not act_f32
     _lib.check(_lib.lib().pg_gated_layernorm_add(y.data_ptr(), y.stride(0), _lib.ptr(gate), 0 if gate is None else gate.stride(0), _lib.ptr(gate_b),
                                                  w1.data_ptr(), b1.data_ptr(), x.data_ptr(), _lib.ptr(w2), _lib.ptr(b2), _lib.ptr(out), rows, D, float(eps),
-                                                 int(ref is not None and ref.dtype == torch.float32), _lib.stream()), "pg_gated_layernorm_add")
+                                                 gate_f32, act_f32, _lib.stream()), "pg_gated_layernorm_add")

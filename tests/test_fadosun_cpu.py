@@ -77,7 +77,8 @@ def test_every_tensor_is_accounted_for_and_the_cache_layout_follows_the_layers()
     del missing["l2.mix.i.b"]
     with pytest.raises(KeyError, match="lacks l2.mix.i.b"):
         model_of(cfg, missing)
-    extra = dict(w, **{"l1.norm2": torch.zeros(24)})  # a layer without a feed-forward has no second norm
+    model_of(cfg, dict(w, **{"l1.norm2": torch.zeros(24)}))  # unused: the layer has no feed-forward
+    extra = dict(w, **{"l1.mlp.up": torch.zeros(20, 24)})
     with pytest.raises(KeyError, match="without a place"):
         model_of(cfg, extra)
     with pytest.raises(ValueError, match="l0.mix.a2"):

@@ -324,6 +324,9 @@ def test_gated_post_norm_residual_and_next_norm(rows, D, f32):
     wide[:, 8:8 + D] = gate.cuda().to(dt)
     seq_ops.gated_layernorm_add(y.cuda(), wide[:, 8:8 + D], dev[0], dev[1], dev[2], x, eps, dev[3], dev[4], out)
     assert worst_row(x, want) < 1e-5 and worst_row(out.float(), O.layer_norm(want, w2, b2, eps)) < (1e-5 if f32 else 1e-2)
+    x = x0.cuda().contiguous()  # an fp32 gate beside either output type
+    seq_ops.gated_layernorm_add(y.cuda(), gate.cuda(), dev[0], dev[1], dev[2], x, eps, dev[3], dev[4], out)
+    assert worst_row(x, want) < 1e-5 and worst_row(out.float(), O.layer_norm(want, w2, b2, eps)) < (1e-5 if f32 else 1e-2)
     x = x0.cuda().contiguous()
     seq_ops.gated_layernorm_add(y.cuda(), gate.cuda().to(dt), dev[0], dev[1], dev[2], x, eps)  # the model's last sub-layer: no norm follows
     assert worst_row(x, want) < 1e-5
