@@ -201,3 +201,10 @@ def test_oracle_whole_equals_prefix():
     tk = torch.randint(0, 30, (20,), generator=torch.Generator().manual_seed(5)).tolist()
     a, b = O.forward(cfg, w, tk), O.forward(cfg, w, tk[:11])
     assert torch.allclose(a[:11], b, atol=1e-9)
+
+
+def test_library_and_host_agree_on_the_normaliser_blocks():
+    from paligemma_multimodal_system_b200 import _lib, build, seq_ops
+    build.build()
+    for v in (1, 4, 7, 16, 24, 64, 128, 130):
+        assert _lib.lib().pg_recurrence_block(v) == seq_ops.recurrence_block(v)
