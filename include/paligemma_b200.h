@@ -327,8 +327,9 @@ int pg_gemm_simt_batched(const void* x, long long ldx, long long batch_x, const 
                          long long ldo, long long batch_out, int tokens, int features, int K, int batch, int in_f32, int out_f32,
                          void* stream);
 
-/* out[t, 0:D] (fp32) = table[tokens[t], col0 : col0 + D] * scale  (embedding lookup; table bf16 or fp32, pitch ld). */
-int pg_embed_rows(const int* tokens, const void* table, long long ld, int col0, float* out, int rows, int D, float scale,
+/* out[t, 0:D] (fp32) = table[tokens[t], col0 : col0 + D] * scale  (embedding lookup; table bf16 or fp32, pitch ld); out_act (may be NULL)
+ * receives the same row in the table's type. */
+int pg_embed_rows(const int* tokens, const void* table, long long ld, int col0, float* out, void* out_act, int rows, int D, float scale,
                   int table_f32, void* stream);
 
 /* Grouped RMS norm folded into the residual add: r = gnorm(y[t, :]) * w, where the row is cut into `groups` equal
@@ -360,11 +361,14 @@ int pg_side_gate(const float* z, long long ldz, const int* tokens, const void* t
  * page_table[row_entry[t] * max_pages + pos[t] / page] * page + pos[t] % page of k_pages [.., G * dim] / v_pages [.., G * vdim].
  * norm_qk == 0 / norm_v == 0 leave out the q/k norm / the value norm; q_norm, k_norm NULL: a norm without a weight; k_pages and
  * v_pages both NULL: the row holds queries only (a layer that attends over another layer's cache).  v_from_k != 0: the row is
- * [q heads | k heads | ...] and value head g is key head g as projected, before norm and rotation (vdim == dim). */
+ * [q heads | k heads | ...] and value head g is key head g as projected, before norm and rotation (vdim == dim).
+ * norm_qk == 2: the norms run over ALL of q (H * dim elements, one mean square, q_norm [H * dim]) and all of k instead of head by head.
+ * rot_gain multiplies every cosine and sine.  v_other != NULL: v <- (1 - v_mix) v + v_mix v_other[t] before it is stored (rows of G * vdim
+ * elements, pitch ld_v_other, activation type). */
 int pg_attn_prepare(const void* qkv, long long ld, const int* pos, const int* row_entry, const int* page_table, int max_pages,
                     int page, const double* freq, const float* q_norm, const float* k_norm, void* q_out, void* k_pages,
                     void* v_pages, int rows, int H, int G, int dim, int vdim, int rot_dims, float eps, int norm_qk, int norm_v, int v_from_k,
-                    int act_f32, void* stream);
+                    float rot_gain, const void* v_other, long long ld_v_other, float v_mix, int act_f32, void* stream);
 
 /* Optional parts of a softmax attention's score and mask, read by pg_attn_ragged, pg_attn_ragged_mma, pg_attn_decode and
  * pg_attn_decode_merge (a NULL pointer or an all-zero struct: plain causal attention).  With i the query's position and j a key's:
@@ -436,13 +440,29 @@ int pg_attn_latent_decode_mma(const void* q, const void* pages, const void* gate
  * per head S <- decay[h] * S + k v^T, out[t, h * vdim + :] = S^T q (fp32).  state: fp32 [slots, H, dim, vdim]; entry e
  * continues state[entry_slot[e]] (from zero when entry_ctx[e] == 0) and leaves its new state there.
  * pg_linear_attn_scan steps token by token; pg_linear_attn_chunked advances in blocks of 32 tokens (same results up to
- * fp32 summation order) and is meant for prompt portions. */
+ * fp32 summation order) and is meant for prompt portions; pg_linear_attn_blocks does so on the tensor cores (bf16, silu == 0, dim <= 128,
+ * dim and vdim multiples of 8, 16-byte aligned rows; every fp32 operand as three bf16 terms).
+ * options (NULL: silu on q, k and v, every entry): silu == 0 -- q and k are turned in pairs (2i, 2i + 1) by the table `rotate` (fp32
+ * [rows, 2, pairs]: cosines, then sines, of the step's rows, made by pg_rotary_table; NULL: not turned), k is multiplied by kscale, and
+ * v is taken as it is, all in fp32; entries with fewer than n_min or more than n_max new tokens are left alone. */
+typedef struct PgLinearAttnOps {
+  int silu;
+  float kscale;
+  const float* rotate;
+  int pairs;
+  int n_min, n_max;
+} PgLinearAttnOps;
+/* out[t, 0, i] = gain * cos(pos[t] * freq[i]), out[t, 1, i] = gain * sin(pos[t] * freq[i]) for i < rot_dims / 2; 1 and 0 for the other pairs. */
+int pg_rotary_table(const int* pos, const double* freq, float* out, int rows, int rot_dims, int pairs, float gain, void* stream);
 int pg_linear_attn_scan(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* entry_row0,
                         const int* entry_n, const int* entry_ctx, const int* entry_slot, int entries, int H, int dim, int vdim,
-                        int act_f32, void* stream);
+                        const PgLinearAttnOps* options, int act_f32, void* stream);
 int pg_linear_attn_chunked(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* entry_row0,
                            const int* entry_n, const int* entry_ctx, const int* entry_slot, int entries, int H, int dim, int vdim,
-                           int act_f32, void* stream);
+                           const PgLinearAttnOps* options, int act_f32, void* stream);
+int pg_linear_attn_blocks(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* entry_row0,
+                          const int* entry_n, const int* entry_ctx, const int* entry_slot, int entries, int H, int dim, int vdim,
+                          const PgLinearAttnOps* options, void* stream);
 
 /* ---- recurrent mixers: a matrix state per head and sequence in fp32 ------------------------------------------------------------
  * Entry e continues slot entry_slot[e] (from zero when entry_ctx[e] == 0) and leaves its new state there.
@@ -511,8 +531,8 @@ int pg_gated_blocks(const PgGatedArgs* args, int kind, int n_min, void* stream);
 int pg_delta_blocks(const PgDeltaArgs* args, float* decay, void* scratch, int max_n, int n_min, void* stream);
 
 /* out[t, :] = scale * G(o[t, :]) with G a norm in `groups` equal consecutive parts (each divided by its own root mean square) times w and a
- * gate: gate_mode 1 -- norm(o) * w * sigmoid(gate); 2 -- norm(o * silu(gate)) * w; 0 -- no gate.  w_n == D: a weight per column;
- * w_n == D / groups: shared by the groups.  o fp32 [rows, D]; gate, out: activation type (pitches ldg, ldo). */
+ * gate: gate_mode 1 -- norm(o) * w * sigmoid(gate); 2 -- norm(o * silu(gate)) * w; 3 -- norm(o) * w * silu(gate); 0 -- no gate.  w_n == D: a
+ * weight per column; w_n == D / groups: shared by the groups; w NULL: no weight.  o fp32 [rows, D]; gate, out: activation type (pitches ldg, ldo). */
 int pg_group_norm_gate(const float* o, const float* w, int w_n, const void* gate, long long ldg, int gate_mode, void* out, long long ldo, int rows,
                        int D, int groups, float eps, float scale, int act_f32, void* stream);
 
@@ -566,16 +586,23 @@ int pg_latent_pack_kv(const void* up, long long ld_up, const void* pages, const 
  *   pair_row[pair] = its sorted row (-1: identity expert).  fill: int32 [n_real] scratch.
  * pg_moe_gemm: out[row, f] = act(sum_k x[src(row), k] * w[expert(row)][f, k]) for the rows of every tile; src(row) =
  *   sorted_pair[row] / src_div when src_div > 0, else row.  w: [n_real] matrices [F, K] (pitch ldw, expert_stride elements apart).
- *   act: 0 none, 2 relu(x)^2, 3 gated silu -- the rows of w alternate gate / up (F even) and out has F / 2 columns:
+ *   act: 0 none, 2 relu(x)^2, 6 gelu (erf form), 3 gated silu -- the rows of w alternate gate / up (F even) and out has F / 2 columns:
  *   out[row, f] = silu(acc[2f]) * acc[2f + 1].  x_expert_off / out_expert_off: elements added to x / out per expert index (0 for routed
  *   experts).  With a host-made plan of (batch index, first row, rows) tiles over the SAME rows for every index this is a batched
  *   product whose operands are column slices: out[:, b, :] = x[:, b, :] w[b]^T (per-head projections on the tensor cores).
  * pg_moe_combine: y[t, :] = sum_k weights[t, k] * (pair_row[t, k] < 0 ? h[t, :] : expert_out[pair_row[t, k], :]) + shared_out[t, :]
  *   (shared_out may be NULL); shared_gate != NULL: the shared term is multiplied by sigmoid(shared_gate[t * ldsg]);
  *   accumulate != 0: y[t, :] += instead of = (y is the fp32 residual stream).
- * pg_moe_route's logit_bias (fp32 [n_all] or NULL) is added to the logits before the softmax. */
+ * pg_moe_route's logit_bias (fp32 [n_all] or NULL) is added to the logits before the softmax.  flags: PG_ROUTE_LOGISTIC -- p = sigmoid(logit)
+ *   instead of the softmax; PG_ROUTE_GROUP_BEST_TWO -- a run's score is the sum of its two largest choices instead of the largest;
+ *   PG_ROUTE_PLAIN_WEIGHTS -- weights[t, k] = p[ids] * scale, not divided by their sum.
+ * pg_moe_combine_norm_add: y = sum_k weights[t, k] * expert_out[pair_row[t, k]] (no identity experts); x[t, :] += y / sqrt(mean(y^2) + eps)
+ *   * norm_w; out_act (may be NULL) gets the new row in the activation type. */
+#define PG_ROUTE_LOGISTIC 1
+#define PG_ROUTE_GROUP_BEST_TWO 2
+#define PG_ROUTE_PLAIN_WEIGHTS 4
 int pg_moe_route(const float* logits, long long ld, const float* correction, int* ids, float* weights, int* counts, int tokens, int n_all,
-                 int n_real, int top, int group_count, int group_keep, float scale, const float* logit_bias, void* stream);
+                 int n_real, int top, int group_count, int group_keep, float scale, const float* logit_bias, int flags, void* stream);
 int pg_moe_tile_rows(void);
 int pg_moe_plan(const int* counts, const int* ids, int* offsets, int* fill, int* plan, int* sorted_pair, int* pair_row, int pairs,
                 int n_real, int max_tiles, void* stream);
@@ -587,14 +614,16 @@ int pg_moe_gemm(const void* x, long long ldx, const int* sorted_pair, int src_di
 int pg_moe_gather_rows(const void* x, long long ldx, const int* sorted_pair, const int* total_rows, int top, void* xg, long long ldg,
                        int max_rows, int D, int act_f32, void* stream);
 /* Per-expert dense products over the gathered runs: expert e owns the next counts_host[e] rows (host array, n_real entries);
- * mid[rows, F] = relu(xg W_up[e]^T)^2 in bf16, eo[rows, D] = mid W_down[e]^T in fp32, both through pg_gemm_bf16.  bf16 only;
- * D, F and the pitches multiples of 8.  glu != 0: w_up holds [n_real, 2F, D] with gate and up rows in blocks of 64
+ * mid[rows, F] = act(xg W_up[e]^T) in bf16, eo[rows, D] = mid W_down[e]^T in fp32, both through pg_gemm_bf16.  bf16 only;
+ * D, F and the pitches multiples of 8.  act: 2 relu(x)^2, 6 gelu (erf form); 3: w_up holds [n_real, 2F, D] with gate and up rows in blocks of 64
  * ([64 gate | 64 up], F a multiple of 64) and mid = silu(gate) * up comes from the product's gated epilogue. */
 int pg_moe_dense_runs(const void* xg, long long ldx, const void* w_up, const void* w_down, void* mid, long long ldm, float* eo, long long ldo,
-                      const int* counts_host, int n_real, int D, int F, int glu, void* stream);
+                      const int* counts_host, int n_real, int D, int F, int act, void* stream);
 int pg_moe_combine(const float* expert_out, long long ldy, const int* pair_row, const int* ids, const float* weights, const void* h,
                    long long ldh, const float* shared_out, long long lds, float* y, int tokens, int D, int top, int act_f32,
                    const float* shared_gate, long long ldsg, int accumulate, void* stream);
+int pg_moe_combine_norm_add(const float* expert_out, long long ldy, const int* pair_row, const float* weights, const float* norm_w, float* x,
+                            void* out_act, int tokens, int D, int top, float eps, int act_f32, void* stream);
 
 #ifdef __cplusplus
 }

@@ -13,7 +13,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("PG_LIB_PATH") or os.path.join(_HERE, "libpaligemma_b200.so")  # PG_LIB_PATH: A/B builds (profiling)
 
 EPI_BF16, EPI_F32, EPI_ATOMIC_F32, EPI_GEGLU = 0, 1, 2, 3
-ABI_VERSION = 5  # pg_abi_version() of the library these signatures describe
+ABI_VERSION = 6  # pg_abi_version() of the library these signatures describe
 
 _ERRORS = {-1: "PG_ERR_ARG", -2: "PG_ERR_CUDA", -3: "PG_ERR_DRIVER", -4: "PG_ERR_TMAP", -5: "PG_ERR_ARCH"}
 
@@ -65,19 +65,21 @@ SIGNATURES = {
     "pg_advance_decode_slots": [p, p, i32, p, p, p, p, i32, p],
     # token-sequence decoders (ragged steps)
     "pg_gemm_simt": [p, i64, p, i64, p, i64, i32, i32, i32, i32, i32, p],
-    "pg_embed_rows": [p, p, i64, i32, p, i32, i32, f32, i32, p],
+    "pg_embed_rows": [p, p, i64, i32, p, p, i32, i32, f32, i32, p],
     "pg_group_rmsnorm_add": [p, i64, p, p, p, i32, i32, i32, f32, i32, p],
     "pg_rmsnorm_gate": [p, p, p, i64, p, i32, i32, f32, i32, p],
     "pg_geglu": [p, i64, p, i64, i32, i32, i32, p],
     "pg_side_gate": [p, i64, p, p, i64, i32, p, i64, i32, i32, i32, i32, p],
-    "pg_attn_prepare": [p, i64, p, p, p, i32, i32, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32, i32, p],
+    "pg_attn_prepare": [p, i64, p, p, p, i32, i32, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, f32, i32, i32, i32, f32, p, i64, f32, i32, p],
     "pg_attn_ragged": [p, p, p, p, i64, p, p, p, p, p, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, i32, i64, i64, i32, p, p],
     "pg_attn_ragged_mma": [p, p, p, p, i64, p, p, p, p, p, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, i32, p, p],
     "pg_attn_decode": [p, p, p, p, i64, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, i64, i64, i32, p, p],
     "pg_attn_decode_merge": [p, p, i64, p, p, p, i32, i32, i32, i32, i32, i32, p, p],
     "pg_attn_latent_decode_mma": [p, p, p, i64, p, p, p, p, p, p, i32, i32, i32, i32, i32, i32, i32, f32, i32, p],
-    "pg_linear_attn_scan": [p, i64, p, p, p, p, p, p, p, i32, i32, i32, i32, i32, p],
-    "pg_linear_attn_chunked": [p, i64, p, p, p, p, p, p, p, i32, i32, i32, i32, i32, p],
+    "pg_linear_attn_scan": [p, i64, p, p, p, p, p, p, p, i32, i32, i32, i32, p, i32, p],
+    "pg_linear_attn_chunked": [p, i64, p, p, p, p, p, p, p, i32, i32, i32, i32, p, i32, p],
+    "pg_linear_attn_blocks": [p, i64, p, p, p, p, p, p, p, i32, i32, i32, i32, p, p],
+    "pg_rotary_table": [p, p, p, i32, i32, i32, f32, p],
     "pg_gemm_simt_batched": [p, i64, i64, p, i64, i64, p, i64, i64, i32, i32, i32, i32, i32, i32, p],
     "pg_embed_streams": [p, p, i64, p, i32, i32, i32, f32, i32, p],
     "pg_stream_mix_norm": [p, p, i64, p, p, p, p, p, i32, i32, i32, f32, i32, p],
@@ -86,7 +88,8 @@ SIGNATURES = {
     "pg_latent_gather": [p, p, i32, i32, p, p, p, p, i32, i32, i32, i32, i32, p],
     "pg_latent_pack_kv": [p, i64, p, p, i32, i32, p, p, p, p, p, i32, i32, i32, i32, i32, i32, i32, i32, p],
     "pg_relu2": [p, i64, i32, i32, i32, p],
-    "pg_moe_route": [p, i64, p, p, p, p, i32, i32, i32, i32, i32, i32, f32, p, p],
+    "pg_moe_route": [p, i64, p, p, p, p, i32, i32, i32, i32, i32, i32, f32, p, i32, p],
+    "pg_moe_combine_norm_add": [p, i64, p, p, p, p, p, i32, i32, i32, f32, i32, p],
     "pg_moe_tile_rows": [],
     "pg_moe_plan": [p, p, p, p, p, p, p, i32, i32, i32, p],
     "pg_moe_gemm": [p, i64, p, i32, p, i64, i64, p, i64, p, i32, i32, i32, i32, i32, i32, i64, i64, p],
@@ -116,6 +119,11 @@ class AttnScore(C.Structure):
     """Mirror of PgAttnScore (include/paligemma_b200.h): the optional parts of an attention's score and mask."""
     _fields_ = [("window", i32), ("keep_first", i32), ("sink", p), ("dist_a", p), ("dist_b", p), ("head_scale", p), ("logistic", i32),
                 ("head_bias", p), ("out_scale", f32), ("out_ld", i64)]
+
+
+class LinearAttnOps(C.Structure):
+    """Mirror of PgLinearAttnOps."""
+    _fields_ = [("silu", i32), ("kscale", f32), ("rotate", p), ("pairs", i32), ("n_min", i32), ("n_max", i32)]
 
 
 class ConvSections(C.Structure):

@@ -38,6 +38,9 @@ PG_DEVINL bool elect_one() {
   return pred != 0;
 }
 
+// 0.5 x (1 + erf(x / sqrt(2)))
+PG_DEVINL float gelu_erf(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)); }
+
 // gelu(tanh) exactly as torch: 0.5 x (1 + tanh( sqrt(2/pi) (x + 0.044715 x^3) ))
 PG_DEVINL float gelu_tanh(float x) {
   const float k0 = 0.7978845608028654f, k1 = 0.044715f;

@@ -129,9 +129,10 @@ PG_DEVINL TileInfo decode_tile(int tile, int m_blocks, int n_blocks, int total_k
   return t;
 }
 
-// activation of the bf16 epilogue (GemmArgs::act_gelu): 1 = gelu(tanh), 2 = relu(x)^2
+// activation of the bf16 epilogue (GemmArgs::act_gelu): 1 = gelu(tanh), 2 = relu(x)^2, 6 = gelu(erf)
 PG_DEVINL float epilogue_act(float x, int act) {
   if (act == 2) { const float r = fmaxf(x, 0.f); return r * r; }
+  if (act == 6) return pg::gelu_erf(x);
   return gelu_tanh_fast(x);
 }
 

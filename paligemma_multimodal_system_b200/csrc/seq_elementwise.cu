@@ -100,13 +100,17 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TI* __restrict__ x
     }
 }
 
-// x[t, :] = table[token[t], col0 : col0 + D] * scale   (fp32 out)
+// x[t, :] = table[token[t], col0 : col0 + D] * scale   (fp32 out; out_act: a copy in the table's type, the first operand of a matrix product)
 template <typename TI>
 __global__ void embed_rows_kernel(const int* __restrict__ tokens, const TI* __restrict__ table, long long ld, int col0, float* __restrict__ out,
-                                  int D, float scale) {
+                                  TI* __restrict__ out_act, int D, float scale) {
   const int t = blockIdx.x;
   const long long row = tokens[t];
-  for (int d = threadIdx.x; d < D; d += blockDim.x) out[(long long)t * D + d] = ld_f(table, row * ld + col0 + d) * scale;
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    const float v = ld_f(table, row * ld + col0 + d) * scale;
+    out[(long long)t * D + d] = v;
+    if (out_act != nullptr) st_f(out_act, (long long)t * D + d, v);
+  }
 }
 
 // Grouped RMS norm of y (fp32) times w, optionally added to the fp32 residual row x (in place); the result (the new residual,
@@ -309,13 +313,13 @@ extern "C" int pg_gemm_simt_batched(const void* x, long long ldx, long long batc
   PG_RET();
 }
 
-extern "C" int pg_embed_rows(const int* tokens, const void* table, long long ld, int col0, float* out, int rows, int D, float scale,
+extern "C" int pg_embed_rows(const int* tokens, const void* table, long long ld, int col0, float* out, void* out_act, int rows, int D, float scale,
                              int table_f32, void* stream) {
   if (rows <= 0 || D <= 0) return PG_ERR_ARG;
   if (table_f32)
-    embed_rows_kernel<float><<<rows, 128, 0, PG_ST(stream)>>>(tokens, static_cast<const float*>(table), ld, col0, out, D, scale);
+    embed_rows_kernel<float><<<rows, 128, 0, PG_ST(stream)>>>(tokens, static_cast<const float*>(table), ld, col0, out, static_cast<float*>(out_act), D, scale);
   else
-    embed_rows_kernel<bf16><<<rows, 128, 0, PG_ST(stream)>>>(tokens, static_cast<const bf16*>(table), ld, col0, out, D, scale);
+    embed_rows_kernel<bf16><<<rows, 128, 0, PG_ST(stream)>>>(tokens, static_cast<const bf16*>(table), ld, col0, out, static_cast<bf16*>(out_act), D, scale);
   PG_RET();
 }
 

@@ -3,13 +3,15 @@
 // already in the paged cache / the recurrent state.  A whole prompt, a portion of one and a single decoded token are
 // the same case with different n and ctx, so the arithmetic of a position never depends on how its sequence was cut.
 //
-//   pg_attn_prepare        q/k RMS norm (shared per-head weight), interleaved partial rotation, weightless value norm;
-//                          k and v rows go to their cache pages, q to a dense buffer
+//   pg_attn_prepare        q/k RMS norm (per head with a shared weight, or over the whole projection), interleaved partial rotation,
+//                          weightless value norm or a blend with another layer's values; k and v rows go to their cache pages, q to a
+//                          dense buffer
 //   pg_attn_ragged         causal softmax (or unnormalised logistic) attention of the new rows over the paged cache (grouped k/v heads,
 //                          tanh soft cap, sigmoid output gate); scores, probabilities and the output accumulation in fp32
 //   pg_linear_attn_scan    decayed outer-product recurrence S <- a S + k v^T, o = S^T q with the state in fp32,
 //                          token by token (decode, short portions)
 //   pg_linear_attn_chunked the same recurrence in blocks of 32 tokens (prompt portions)
+//                          (both: q, k, v through silu, or q and k rotated and k scaled, in fp32 as they are read)
 #include "common.cuh"
 #include "paligemma_b200.h"
 
@@ -60,21 +62,36 @@ __global__ void __launch_bounds__(128) attn_prepare_kernel(const TA* __restrict_
                                                            int page, const double* __restrict__ freq, const float* __restrict__ qn,
                                                            const float* __restrict__ kn, TA* __restrict__ q_out, TA* __restrict__ k_pages,
                                                            TA* __restrict__ v_pages, int H, int G, int dim, int vdim, int rot, float eps,
-                                                           int norm_qk, int norm_v, int v_from_k) {
+                                                           int norm_qk, int norm_v, int v_from_k, float rot_gain,
+                                                           const TA* __restrict__ v_other, long long ldvo, float v_mix) {
   extern __shared__ float cs[];  // cos[rot/2], sin[rot/2]
   const long long t = blockIdx.x;
   const int p = pos[t];
   for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
     double s, c;
     sincos((double)p * freq[i], &s, &c);
-    cs[i] = (float)c;
-    cs[rot / 2 + i] = (float)s;
+    cs[i] = rot_gain * (float)c;
+    cs[rot / 2 + i] = rot_gain * (float)s;
   }
   __syncthreads();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const long long pg_row = (long long)page_table[(long long)row_entry[t] * max_pages + p / page] * page + p % page;
   const TA* row = qkv + t * ld;
   const int nvec = k_pages != nullptr ? H + 2 * G : H;  // a layer that borrows another layer's keys / values prepares its queries only
+  float inv_q = 1.0f, inv_k = 1.0f;
+  if (norm_qk == 2) {  // one root mean square for all of q, one for all of k
+    __shared__ float part[2][4];
+    const int nq = H * dim, nk = k_pages != nullptr ? G * dim : 0;
+    float sq = 0.f, sk = 0.f;
+    for (int d = threadIdx.x; d < nq; d += 128) { const float a = ldf(row, d); sq = fmaf(a, a, sq); }
+    for (int d = threadIdx.x; d < nk; d += 128) { const float a = ldf(row, (long long)nq + d); sk = fmaf(a, a, sk); }
+    sq = wsum(sq);
+    sk = wsum(sk);
+    if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
+    __syncthreads();
+    inv_q = 1.0f / sqrtf((part[0][0] + part[0][1] + part[0][2] + part[0][3]) / (float)nq + eps);
+    if (nk > 0) inv_k = 1.0f / sqrtf((part[1][0] + part[1][1] + part[1][2] + part[1][3]) / (float)nk + eps);
+  }
   for (int vec = warp; vec < nvec; vec += nw) {
     const bool is_q = vec < H, is_k = !is_q && vec < H + G;
     const int n = (is_q || is_k) ? dim : vdim;
@@ -83,8 +100,8 @@ __global__ void __launch_bounds__(128) attn_prepare_kernel(const TA* __restrict_
                           : v_from_k ? (long long)H * dim + (long long)(vec - H - G) * dim
                                      : (long long)(H + G) * dim + (long long)(vec - H - G) * vdim;
     // lane <-> pairs (2i, 2i+1): a rotation never needs another lane's element; an odd last element is a pair with a zero
-    float inv = 1.0f;
-    if ((is_q || is_k) ? norm_qk : norm_v) {
+    float inv = is_q ? inv_q : is_k ? inv_k : 1.0f;
+    if ((is_q || is_k) ? norm_qk == 1 : norm_v) {
       float ss = 0.f;
       for (int d = 2 * lane; d < n; d += 64) {
         const float a = ldf(row, off + d), b2 = d + 1 < n ? ldf(row, off + d + 1) : 0.f;
@@ -94,6 +111,8 @@ __global__ void __launch_bounds__(128) attn_prepare_kernel(const TA* __restrict_
       inv = 1.0f / sqrtf(ss / (float)n + eps);
     }
     const float* w = is_q ? qn : kn;  // NULL: a norm without a weight
+    if (norm_qk == 2 && w != nullptr) w += (long long)(is_q ? vec : vec - H) * dim;
+    const TA* vo = (v_other != nullptr && !is_q && !is_k) ? v_other + t * ldvo + (long long)(vec - H - G) * vdim : nullptr;
     TA* dst = is_q   ? q_out + t * ((long long)H * dim) + (long long)vec * dim
               : is_k ? k_pages + pg_row * ((long long)G * dim) + (long long)(vec - H) * dim
                      : v_pages + pg_row * ((long long)G * vdim) + (long long)(vec - H - G) * vdim;
@@ -110,6 +129,9 @@ __global__ void __launch_bounds__(128) attn_prepare_kernel(const TA* __restrict_
           const float ra = a * c - b2 * sn, rb = b2 * c + a * sn;
           a = ra; b2 = rb;
         }
+      } else if (vo != nullptr) {
+        a = (1.0f - v_mix) * a + v_mix * ldf(vo, d);
+        if (two) b2 = (1.0f - v_mix) * b2 + v_mix * ldf(vo, d + 1);
       }
       stf(dst, d, a);
       if (two) stf(dst, d + 1, b2);
@@ -560,14 +582,27 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ partial, cons
 // column x one slice of DC key dimensions, its part of the state in registers.  q, k, v = silu(projection) are formed
 // in fp32 from the activation-type projections; state, decay and output are fp32.
 // ---------------------------------------------------------------------------------------------------------------------
+// A projected q / k pair (elements 2 i, 2 i + 1 of a head) on its way into a recurrence without silu: the rotation by the row's cosines and
+// sines (table row: `pairs` cosines, then `pairs` sines; 1 and 0 past the rotated pairs; NULL: none), then a factor.
+__device__ __forceinline__ void enter_pair(const PgLinearAttnOps& ops, long long t, int i, float factor, float& a, float& b) {
+  if (ops.rotate != nullptr) {
+    const float c = ops.rotate[t * 2 * ops.pairs + i], s = ops.rotate[(t * 2 + 1) * ops.pairs + i];
+    const float ra = a * c - b * s, rb = b * c + a * s;
+    a = ra; b = rb;
+  }
+  a *= factor;
+  b *= factor;
+}
+
 template <typename TA, int DCMAX>
 __global__ void __launch_bounds__(256) linear_attn_scan_kernel(const TA* __restrict__ qkv, long long ld, float* __restrict__ state,
                                                                const float* __restrict__ decay, float* __restrict__ out,
                                                                const int* __restrict__ entry_row0, const int* __restrict__ entry_n,
                                                                const int* __restrict__ entry_ctx, const int* __restrict__ entry_slot, int H,
-                                                               int dim, int vdim, int VB) {
+                                                               int dim, int vdim, int VB, PgLinearAttnOps ops) {
   const int e = blockIdx.z, h = blockIdx.y, vb = blockIdx.x;
   const int n = entry_n[e], row0 = entry_row0[e];
+  if (n < ops.n_min || n > ops.n_max) return;
   const int nchunk = 256 / VB, DC = (dim + nchunk - 1) / nchunk;
   const int vl = threadIdx.x % VB, chunk = threadIdx.x / VB;
   const int v = vb * VB + vl;
@@ -588,11 +623,25 @@ __global__ void __launch_bounds__(256) linear_attn_scan_kernel(const TA* __restr
   const long long qo = (long long)h * dim, ko = (long long)H * dim + (long long)h * dim, vo = 2LL * H * dim + (long long)h * vdim;
   for (int t = 0; t < n; ++t) {
     const TA* row = qkv + (long long)(row0 + t) * ld;
-    for (int d = threadIdx.x; d < dim; d += 256) {
-      qs[d] = silu(ldf(row, qo + d));
-      ksm[d] = silu(ldf(row, ko + d));
+    float vv = v_ok ? ldf(row, vo + v) : 0.f;
+    if (ops.silu) {
+      for (int d = threadIdx.x; d < dim; d += 256) {
+        qs[d] = silu(ldf(row, qo + d));
+        ksm[d] = silu(ldf(row, ko + d));
+      }
+      vv = silu(vv);
+    } else {
+      for (int i = threadIdx.x; 2 * i < dim; i += 256) {
+        const int d = 2 * i;
+        const bool two = d + 1 < dim;
+        float q0 = ldf(row, qo + d), q1 = two ? ldf(row, qo + d + 1) : 0.f, k0 = ldf(row, ko + d), k1 = two ? ldf(row, ko + d + 1) : 0.f;
+        enter_pair(ops, row0 + t, i, 1.0f, q0, q1);
+        enter_pair(ops, row0 + t, i, ops.kscale, k0, k1);
+        qs[d] = q0;
+        ksm[d] = k0;
+        if (two) { qs[d + 1] = q1; ksm[d + 1] = k1; }
+      }
     }
-    const float vv = v_ok ? silu(ldf(row, vo + v)) : 0.f;
     __syncthreads();
     float part = 0.f;
 #pragma unroll
@@ -631,10 +680,11 @@ __global__ void __launch_bounds__(256, 2) linear_attn_chunked_kernel(const TA* _
                                                                   const float* __restrict__ decay, float* __restrict__ out,
                                                                   const int* __restrict__ entry_row0, const int* __restrict__ entry_n,
                                                                   const int* __restrict__ entry_ctx, const int* __restrict__ entry_slot, int H,
-                                                                  int dim, int vdim) {
+                                                                  int dim, int vdim, PgLinearAttnOps ops) {
   constexpr int C = 32;
   const int e = blockIdx.z, h = blockIdx.y, vb = blockIdx.x;
   const int n = entry_n[e], row0 = entry_row0[e];
+  if (n < ops.n_min || n > ops.n_max) return;
   constexpr int ngrp = 256 / VB, rpt = C / ngrp;  // row groups; rows per thread (8 for 64 value columns per CTA)
   const int vl = threadIdx.x % VB, grp = threadIdx.x / VB;  // a warp lies inside one group: its row / key operands are broadcasts
   const int v = vb * VB + vl;
@@ -690,34 +740,49 @@ __global__ void __launch_bounds__(256, 2) linear_attn_chunked_kernel(const TA* _
       for (int k = 0; k < 2; ++k) {
         const int idx = threadIdx.x + 256 * k, r = idx / d8, c = (idx % d8) * 8;
         if (idx < C * d8) {
+          if (!ops.silu && r < cn) {
+#pragma unroll
+            for (int x = 0; x < 8; x += 2) {
+              enter_pair(ops, row0 + t0 + r, (c + x) / 2, 1.0f, pq[k][x], pq[k][x + 1]);
+              enter_pair(ops, row0 + t0 + r, (c + x) / 2, ops.kscale, pk[k][x], pk[k][x + 1]);
+            }
+          }
 #pragma unroll
           for (int x = 0; x < 8; ++x) {
-            Qs[r * kd + c + x] = act(pq[k][x]);
-            Ks[r * kd + c + x] = act(pk[k][x]);
+            Qs[r * kd + c + x] = ops.silu ? act(pq[k][x]) : pq[k][x];
+            Ks[r * kd + c + x] = ops.silu ? act(pk[k][x]) : pk[k][x];
           }
         }
       }
       if (threadIdx.x < C * v8) {
         const int r = threadIdx.x / v8, c = (threadIdx.x % v8) * 8;
 #pragma unroll
-        for (int x = 0; x < 8; ++x) Vs[r * VB + c + x] = act(pv[x]);
+        for (int x = 0; x < 8; ++x) Vs[r * VB + c + x] = ops.silu ? act(pv[x]) : pv[x];
       }
       if (t0 + C < n) fetch(t0 + C);
     } else {
-      for (int i = threadIdx.x; i < C * dim4; i += 256) {
-        const int r = i / dim4, d = i % dim4;
-        float qv = 0.f, kv = 0.f;
+      for (int i = threadIdx.x; i < C * dim4 / 2; i += 256) {
+        const int r = i / (dim4 / 2), p2 = i % (dim4 / 2), d = 2 * p2;
+        float q0 = 0.f, q1 = 0.f, k0 = 0.f, k1 = 0.f;
         if (r < cn && d < dim) {
           const TA* row = qkv + (long long)(row0 + t0 + r) * ld;
-          qv = silu(ldf(row, qo + d));
-          kv = silu(ldf(row, ko + d));
+          const bool two = d + 1 < dim;
+          q0 = ldf(row, qo + d); k0 = ldf(row, ko + d);
+          if (two) { q1 = ldf(row, qo + d + 1); k1 = ldf(row, ko + d + 1); }
+          if (ops.silu) {
+            q0 = silu(q0); q1 = silu(q1); k0 = silu(k0); k1 = silu(k1);
+          } else {
+            enter_pair(ops, row0 + t0 + r, p2, 1.0f, q0, q1);
+            enter_pair(ops, row0 + t0 + r, p2, ops.kscale, k0, k1);
+          }
         }
-        Qs[r * kd + d] = qv;
-        Ks[r * kd + d] = kv;
+        Qs[r * kd + d] = q0; Qs[r * kd + d + 1] = q1;
+        Ks[r * kd + d] = k0; Ks[r * kd + d + 1] = k1;
       }
       for (int i = threadIdx.x; i < C * VB; i += 256) {
         const int r = i / VB, c = vb * VB + i % VB;
-        Vs[i] = (r < cn && c < vdim) ? silu(ldf(qkv + (long long)(row0 + t0 + r) * ld, vo + c)) : 0.f;
+        const float raw = (r < cn && c < vdim) ? ldf(qkv + (long long)(row0 + t0 + r) * ld, vo + c) : 0.f;
+        Vs[i] = ops.silu ? silu(raw) : raw;
       }
     }
     __syncthreads();
@@ -795,22 +860,50 @@ __global__ void __launch_bounds__(256, 2) linear_attn_chunked_kernel(const TA* _
 
 }  // namespace
 
+// out[t, 0, i] = gain cos(pos[t] freq[i]), out[t, 1, i] = gain sin(.) for i < rot / 2; 1 and 0 for the other pairs
+__global__ void rotary_table_kernel(const int* __restrict__ pos, const double* __restrict__ freq, float* __restrict__ out, int rot, int pairs, float gain,
+                                    long long total) {
+  const long long id = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (id >= total) return;
+  const long long t = id / pairs;
+  const int i = (int)(id % pairs);
+  float c = 1.0f, s = 0.0f;
+  if (2 * i < rot) {
+    double sd, cd;
+    sincos((double)pos[t] * freq[i], &sd, &cd);
+    c = gain * (float)cd;
+    s = gain * (float)sd;
+  }
+  out[t * 2 * pairs + i] = c;
+  out[(t * 2 + 1) * pairs + i] = s;
+}
+
+extern "C" int pg_rotary_table(const int* pos, const double* freq, float* out, int rows, int rot_dims, int pairs, float gain, void* stream) {
+  if (rows <= 0 || rot_dims < 0 || (rot_dims & 1) || pairs <= 0 || 2 * pairs < rot_dims) return PG_ERR_ARG;
+  const long long total = (long long)rows * pairs;
+  rotary_table_kernel<<<(unsigned)((total + 127) / 128), 128, 0, PG_ST(stream)>>>(pos, freq, out, rot_dims, pairs, gain, total);
+  PG_RET();
+}
+
 extern "C" int pg_attn_prepare(const void* qkv, long long ld, const int* pos, const int* row_entry, const int* page_table, int max_pages,
                                int page, const double* freq, const float* q_norm, const float* k_norm, void* q_out, void* k_pages,
                                void* v_pages, int rows, int H, int G, int dim, int vdim, int rot_dims, float eps, int norm_qk, int norm_v,
-                               int v_from_k, int act_f32, void* stream) {
+                               int v_from_k, float rot_gain, const void* v_other, long long ld_v_other, float v_mix, int act_f32, void* stream) {
   if (rows <= 0 || H <= 0 || G <= 0 || dim <= 0 || vdim <= 0 || rot_dims < 0 || rot_dims > dim || (rot_dims & 1) || page <= 0) return PG_ERR_ARG;
   if (v_from_k && vdim != dim) return PG_ERR_ARG;
+  if (norm_qk < 0 || norm_qk > 2 || (v_other != nullptr && k_pages == nullptr)) return PG_ERR_ARG;
   if ((k_pages == nullptr) != (v_pages == nullptr)) return PG_ERR_ARG;
   const size_t smem = (size_t)(rot_dims + 2) * sizeof(float);
   if (act_f32)
     attn_prepare_kernel<float><<<rows, 128, smem, PG_ST(stream)>>>(static_cast<const float*>(qkv), ld, pos, row_entry, page_table, max_pages, page, freq,
                                                                   q_norm, k_norm, static_cast<float*>(q_out), static_cast<float*>(k_pages),
-                                                                  static_cast<float*>(v_pages), H, G, dim, vdim, rot_dims, eps, norm_qk, norm_v, v_from_k);
+                                                                  static_cast<float*>(v_pages), H, G, dim, vdim, rot_dims, eps, norm_qk, norm_v, v_from_k, rot_gain,
+                                                                  static_cast<const float*>(v_other), ld_v_other, v_mix);
   else
     attn_prepare_kernel<bf16><<<rows, 128, smem, PG_ST(stream)>>>(static_cast<const bf16*>(qkv), ld, pos, row_entry, page_table, max_pages, page, freq,
                                                                  q_norm, k_norm, static_cast<bf16*>(q_out), static_cast<bf16*>(k_pages),
-                                                                 static_cast<bf16*>(v_pages), H, G, dim, vdim, rot_dims, eps, norm_qk, norm_v, v_from_k);
+                                                                 static_cast<bf16*>(v_pages), H, G, dim, vdim, rot_dims, eps, norm_qk, norm_v, v_from_k, rot_gain,
+                                                                 static_cast<const bf16*>(v_other), ld_v_other, v_mix);
   PG_RET();
 }
 
@@ -860,26 +953,34 @@ extern "C" int pg_attn_ragged(const void* q, const void* k_pages, const void* v_
 #undef PG_ATTN
 }
 
+// NULL: silu on q, k and v, entries of any length
+static bool linear_attn_ops(const PgLinearAttnOps* options, int dim, PgLinearAttnOps& ops) {
+  ops = options != nullptr ? *options : PgLinearAttnOps{1, 1.0f, nullptr, 0, 1, 0x7fffffff};
+  return ops.rotate == nullptr || (!ops.silu && 2 * ops.pairs >= dim);
+}
+
 template <typename TA, int DCMAX>
 static int launch_scan(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* row0, const int* n, const int* ctx,
-                       const int* slot, int entries, int H, int dim, int vdim, int VB, cudaStream_t st) {
+                       const int* slot, int entries, int H, int dim, int vdim, int VB, const PgLinearAttnOps& ops, cudaStream_t st) {
   const int nchunk = 256 / VB;
   const size_t smem = ((size_t)2 * dim + (size_t)nchunk * VB) * sizeof(float);
   dim3 grid((vdim + VB - 1) / VB, H, entries);
-  linear_attn_scan_kernel<TA, DCMAX><<<grid, 256, smem, st>>>(static_cast<const TA*>(qkv), ld, state, decay, out, row0, n, ctx, slot, H, dim, vdim, VB);
+  linear_attn_scan_kernel<TA, DCMAX><<<grid, 256, smem, st>>>(static_cast<const TA*>(qkv), ld, state, decay, out, row0, n, ctx, slot, H, dim, vdim, VB, ops);
   PG_RET();
 }
 
 extern "C" int pg_linear_attn_scan(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* entry_row0,
                                    const int* entry_n, const int* entry_ctx, const int* entry_slot, int entries, int H, int dim, int vdim,
-                                   int act_f32, void* stream) {
+                                   const PgLinearAttnOps* options, int act_f32, void* stream) {
   if (entries <= 0 || H <= 0 || dim <= 0 || vdim <= 0 || dim > 1024 || entries > 65535 || H > 65535) return PG_ERR_ARG;
+  PgLinearAttnOps ops;
+  if (!linear_attn_ops(options, dim, ops)) return PG_ERR_ARG;
   cudaStream_t st = PG_ST(stream);
   // VB value columns per CTA (a power of two <= 64); the 256 / VB thread groups split the key dimensions
   int VB = 64;
   while (VB > 8 && VB / 2 >= vdim) VB /= 2;
   const int DC = (dim + 256 / VB - 1) / (256 / VB);
-#define PG_SCAN(TA, DCM) return launch_scan<TA, DCM>(qkv, ld, state, decay, out, entry_row0, entry_n, entry_ctx, entry_slot, entries, H, dim, vdim, VB, st)
+#define PG_SCAN(TA, DCM) return launch_scan<TA, DCM>(qkv, ld, state, decay, out, entry_row0, entry_n, entry_ctx, entry_slot, entries, H, dim, vdim, VB, ops, st)
   if (act_f32) {
     if (DC <= 16) PG_SCAN(float, 16);
     if (DC <= 64) PG_SCAN(float, 64);
@@ -893,17 +994,19 @@ extern "C" int pg_linear_attn_scan(const void* qkv, long long ld, float* state, 
 
 template <typename TA, bool VEC, int VB>
 static int launch_chunked(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* row0, const int* n, const int* ctx,
-                          const int* slot, int entries, int H, int dim, int vdim, size_t smem, cudaStream_t st) {
+                          const int* slot, int entries, int H, int dim, int vdim, size_t smem, const PgLinearAttnOps& ops, cudaStream_t st) {
   auto kern = linear_attn_chunked_kernel<TA, VEC, VB>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return PG_ERR_CUDA;
-  kern<<<dim3((vdim + VB - 1) / VB, H, entries), 256, smem, st>>>(static_cast<const TA*>(qkv), ld, state, decay, out, row0, n, ctx, slot, H, dim, vdim);
+  kern<<<dim3((vdim + VB - 1) / VB, H, entries), 256, smem, st>>>(static_cast<const TA*>(qkv), ld, state, decay, out, row0, n, ctx, slot, H, dim, vdim, ops);
   PG_RET();
 }
 
 extern "C" int pg_linear_attn_chunked(const void* qkv, long long ld, float* state, const float* decay, float* out, const int* entry_row0,
                                       const int* entry_n, const int* entry_ctx, const int* entry_slot, int entries, int H, int dim, int vdim,
-                                      int act_f32, void* stream) {
+                                      const PgLinearAttnOps* options, int act_f32, void* stream) {
   if (entries <= 0 || H <= 0 || dim <= 0 || vdim <= 0 || entries > 65535 || H > 65535) return PG_ERR_ARG;
+  PgLinearAttnOps ops;
+  if (!linear_attn_ops(options, dim, ops)) return PG_ERR_ARG;
   int VB = 64;
   while (VB > 8 && VB / 2 >= vdim) VB /= 2;
   // narrower value blocks (the scores are recomputed per block) only while the grid does not even fill the SMs once
@@ -917,7 +1020,7 @@ extern "C" int pg_linear_attn_chunked(const void* qkv, long long ld, float* stat
   // 16-byte fetches: every head's q / k / v slice of a row starts on an 8-element boundary
   const bool vec = dim % 8 == 0 && vdim % 8 == 0 && dim <= 128 && ld % 8 == 0 && (reinterpret_cast<uintptr_t>(qkv) & 15) == 0;
 #define PG_CHUNK(TA, VEC, VBV) \
-  return launch_chunked<TA, VEC, VBV>(qkv, ld, state, decay, out, entry_row0, entry_n, entry_ctx, entry_slot, entries, H, dim, vdim, smem, st)
+  return launch_chunked<TA, VEC, VBV>(qkv, ld, state, decay, out, entry_row0, entry_n, entry_ctx, entry_slot, entries, H, dim, vdim, smem, ops, st)
 #define PG_CHUNK_VB(TA, VEC)          \
   do {                                \
     if (VB == 64) PG_CHUNK(TA, VEC, 64); \

@@ -1,14 +1,15 @@
 // Routed feed-forward (mixture of experts) of the token-sequence decoders, without a host round trip: the step may sit in a
 // CUDA graph, so counts, offsets and tile lists stay on the device.
 //
-//   pg_moe_route     per token: softmax over the router outputs, choice score = probability + correction, optional group limit
-//                    (experts in `group_count` equal runs of neighbours; only the `group_keep` runs with the largest best
-//                    choice score stay eligible), the `top` largest choice scores, weights = chosen probabilities / their sum
-//                    * scale.  Outputs >= n_real are identity experts.  Counts the (token, choice) pairs of every real expert.
+//   pg_moe_route     per token: scores = softmax over the router outputs (or their logistic function), choice score = score + correction,
+//                    optional group limit (experts in `group_count` equal runs of neighbours; only the `group_keep` runs with the
+//                    largest best choice score, or sum of the two best, stay eligible), the `top` largest choice scores, weights =
+//                    chosen scores (/ their sum) * scale.  Outputs >= n_real are identity experts.  Counts the (token, choice) pairs of every real expert.
 //   pg_moe_plan      one CTA: expert offsets (exclusive scan), the list of row tiles (expert, first row, rows) and its length
 //   pg_moe_scatter   pair -> its row in the expert-sorted order (and back)
 //   pg_moe_gemm      out[row, f] = act(sum_k x[src(row), k] w[expert(row)][f, k]) over the tile list; plain fp32 FMAs, or
 //                    mma.sync on the tensor cores for bf16 operands
+//   pg_moe_combine_norm_add  the same sum, its norm and the residual add in one pass
 //   pg_moe_combine   y[t] = sum_k weight[t, k] * (identity ? h[t] : expert_out[row(t, k)]) (+ shared[t])
 //
 // Router arithmetic, weights and the combine are fp32.
@@ -61,7 +62,7 @@ __device__ __forceinline__ void wargmax(float& v, int& i) {
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction,
                                                         int* __restrict__ ids, float* __restrict__ weights, int* __restrict__ counts, int T,
                                                         int n_all, int n_real, int top, int group_count, int group_keep, float scale,
-                                                        const float* __restrict__ logit_bias) {
+                                                        const float* __restrict__ logit_bias, int flags) {
   extern __shared__ float sm[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x * 4 + warp;
@@ -75,28 +76,34 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     prob[i] = zi;
     m = fmaxf(m, zi);
   }
-  m = wmaxf(m);
   float s = 0.f;
-  for (int i = lane; i < n_all; i += 32) { const float e = expf(prob[i] - m); prob[i] = e; s += e; }
-  s = wsumf(s);
+  if (!(flags & PG_ROUTE_LOGISTIC)) {
+    m = wmaxf(m);
+    for (int i = lane; i < n_all; i += 32) { const float e = expf(prob[i] - m); prob[i] = e; s += e; }
+    s = wsumf(s);
+  }
   for (int i = lane; i < n_all; i += 32) {
-    const float p = prob[i] / s;
+    const float p = (flags & PG_ROUTE_LOGISTIC) ? 1.0f / (1.0f + expf(-prob[i])) : prob[i] / s;
     prob[i] = p;
     choice[i] = p + (correction != nullptr ? correction[i] : 0.f);
   }
   __syncwarp();
   if (group_count > 1 && group_keep < group_count) {
-    // group g lives in lane g % 32, slot g / 32 (up to 8 slots = 256 groups): its score is its best choice score; group_keep rounds of
-    // a warp arg-max mark the kept groups, the others get -inf choice scores (not 0: choice scores can be negative)
+    // group g lives in lane g % 32, slot g / 32 (up to 8 slots = 256 groups): its score is its best choice score (or the sum of the two
+    // best); group_keep rounds of a warp arg-max mark the kept groups, the others get -inf choice scores (not 0: choice scores can be negative)
     const int per = n_all / group_count;
     float gs[8];
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
       const int g = lane + 32 * k;
-      float b = -INFINITY;
+      float b = -INFINITY, second = -INFINITY;
       if (g < group_count)
-        for (int i = 0; i < per; ++i) b = fmaxf(b, choice[g * per + i]);
-      gs[k] = b;
+        for (int i = 0; i < per; ++i) {
+          const float c = choice[g * per + i];
+          second = fmaxf(second, fminf(b, c));
+          b = fmaxf(b, c);
+        }
+      gs[k] = ((flags & PG_ROUTE_GROUP_BEST_TWO) && per > 1) ? b + second : b;
     }
     unsigned keepmask[8] = {0, 0, 0, 0, 0, 0, 0, 0};  // slot k kept (meaningful in the owning lane only)
     for (int r = 0; r < group_keep; ++r) {
@@ -141,38 +148,49 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
       const int base = r & ~31;
       if (my_id >= 0) {
         ids[(long long)t * top + base + lane] = my_id;
-        weights[(long long)t * top + base + lane] = my_p;  // normalised below
+        weights[(long long)t * top + base + lane] = my_p;  // scaled below
         if (my_id < n_real) atomicAdd(counts + my_id, 1);
       }
       my_id = -1;
     }
   }
   __syncwarp();
-  const float f = scale / (wsum_sel + 1e-20f);
+  const float f = (flags & PG_ROUTE_PLAIN_WEIGHTS) ? scale : scale / (wsum_sel + 1e-20f);
   for (int r = lane; r < top; r += 32) weights[(long long)t * top + r] *= f;
 }
 
 // counts -> offsets, tile list.  plan[0] = number of tiles; tiles: (expert, first sorted row, rows) triples from plan[4].
+// One warp: 32 experts at a time, prefix sums of their counts and tile numbers by shuffles.
 __global__ void moe_plan_kernel(const int* __restrict__ counts, int* __restrict__ offsets, int* __restrict__ fill, int* __restrict__ plan, int n_real,
                                 int max_tiles) {
-  if (threadIdx.x != 0) return;
+  const int lane = threadIdx.x;
   int off = 0, nt = 0;
-  for (int e = 0; e < n_real; ++e) {
-    const int c = counts[e];
-    offsets[e] = off;
-    fill[e] = 0;
-    for (int r = 0; r < c; r += MOE_TILE) {
-      if (nt < max_tiles) {
-        plan[4 + 3 * nt] = e;
-        plan[4 + 3 * nt + 1] = off + r;
-        plan[4 + 3 * nt + 2] = min(MOE_TILE, c - r);
-      }
-      ++nt;
+  for (int e0 = 0; e0 < n_real; e0 += 32) {
+    const int e = e0 + lane, c = e < n_real ? counts[e] : 0, tiles = (c + MOE_TILE - 1) / MOE_TILE;
+    int pc = c, ptl = tiles;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int a = __shfl_up_sync(0xffffffffu, pc, o), b = __shfl_up_sync(0xffffffffu, ptl, o);
+      if (lane >= o) { pc += a; ptl += b; }
     }
-    off += c;
+    const int first = off + pc - c, tile0 = nt + ptl - tiles;
+    if (e < n_real) {
+      offsets[e] = first;
+      fill[e] = 0;
+    }
+    for (int r = 0; r < tiles && tile0 + r < max_tiles; ++r) {
+      int* p = plan + 4 + 3 * (tile0 + r);
+      p[0] = e;
+      p[1] = first + r * MOE_TILE;
+      p[2] = min(MOE_TILE, c - r * MOE_TILE);
+    }
+    off += __shfl_sync(0xffffffffu, pc, 31);
+    nt += __shfl_sync(0xffffffffu, ptl, 31);
   }
-  offsets[n_real] = off;
-  plan[0] = nt < max_tiles ? nt : max_tiles;
+  if (lane == 0) {
+    offsets[n_real] = off;
+    plan[0] = nt < max_tiles ? nt : max_tiles;
+  }
 }
 
 __global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __restrict__ offsets, int* __restrict__ fill, int* __restrict__ sorted_pair,
@@ -253,6 +271,7 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TI* __restrict__ x,
       if (r < nr && f < F) {
         float v = acc[i][j];
         if (act == 2) { v = fmaxf(v, 0.f); v *= v; }
+        if (act == 6) v = pg::gelu_erf(v);
         stm(out, (long long)(r0 + r) * ldo + f, v);
       }
     }
@@ -383,6 +402,7 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(const bf16* __restric
         if (r < nr && f < F) {
           float v = acc[mi][ni][c];
           if (act == 2) { v = fmaxf(v, 0.f); v *= v; }
+          if (act == 6) v = pg::gelu_erf(v);
           stm(out, (long long)(r0 + r) * ldo + f, v);
         }
       }
@@ -432,10 +452,84 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, long lo
   }
 }
 
+// The combine, a norm of its result and the residual add in one pass: y = sum_k weights[t, k] * expert row,
+// x[t] += y / rms(y) * w, and a copy of the new x in the activation type.  One CTA per row; y stays in shared memory.  VEC: 16-byte accesses.
+template <typename TA, bool VEC>
+__global__ void __launch_bounds__(256) moe_combine_norm_add_kernel(const float* __restrict__ expert_out, long long ldy, const int* __restrict__ pair_row,
+                                                                   const float* __restrict__ weights, const float* __restrict__ norm_w,
+                                                                   float* __restrict__ x, TA* __restrict__ out_act, int D, int top, float eps) {
+  extern __shared__ __align__(16) float comb_y[];  // [D]
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float s = 0.f;
+  if (VEC) {
+    for (int d = threadIdx.x; d < D / 4; d += 256) {
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+      for (int k = 0; k < top; ++k) {
+        const float g = weights[t * top + k];
+        const float4 v = reinterpret_cast<const float4*>(expert_out + (long long)pair_row[t * top + k] * ldy)[d];
+        a.x = fmaf(g, v.x, a.x); a.y = fmaf(g, v.y, a.y); a.z = fmaf(g, v.z, a.z); a.w = fmaf(g, v.w, a.w);
+      }
+      reinterpret_cast<float4*>(comb_y)[d] = a;
+      s = fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, s))));
+    }
+  } else {
+    for (int d = threadIdx.x; d < D; d += 256) {
+      float a = 0.f;
+      for (int k = 0; k < top; ++k) a = fmaf(weights[t * top + k], expert_out[(long long)pair_row[t * top + k] * ldy + d], a);
+      comb_y[d] = a;
+      s = fmaf(a, a, s);
+    }
+  }
+  s = wsumf(s);
+  if (lane == 0) red[warp] = s;
+  __syncthreads();
+  s = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) s += red[w];
+  const float inv = 1.0f / sqrtf(s / (float)D + eps);
+  // a thread reads back the elements it wrote
+  if (VEC) {
+    for (int d = threadIdx.x; d < D / 4; d += 256) {
+      const float4 a = reinterpret_cast<const float4*>(comb_y)[d], w = reinterpret_cast<const float4*>(norm_w)[d];
+      float4* xp = reinterpret_cast<float4*>(x + t * D) + d;
+      float4 v = *xp;
+      v.x += a.x * inv * w.x; v.y += a.y * inv * w.y; v.z += a.z * inv * w.z; v.w += a.w * inv * w.w;
+      *xp = v;
+      if (out_act != nullptr) {
+        if constexpr (sizeof(TA) == 4) *reinterpret_cast<float4*>(out_act + t * D + 4 * d) = v;
+        else *reinterpret_cast<uint2*>(out_act + t * D + 4 * d) = make_uint2(pg::pack_bf16(v.x, v.y), pg::pack_bf16(v.z, v.w));
+      }
+    }
+  } else {
+    for (int d = threadIdx.x; d < D; d += 256) {
+      const float v = x[t * D + d] + comb_y[d] * inv * norm_w[d];
+      x[t * D + d] = v;
+      if (out_act != nullptr) stm(out_act, t * D + d, v);
+    }
+  }
+}
+
 }  // namespace
 
+extern "C" int pg_moe_combine_norm_add(const float* expert_out, long long ldy, const int* pair_row, const float* weights, const float* norm_w, float* x,
+                                       void* out_act, int tokens, int D, int top, float eps, int act_f32, void* stream) {
+  if (tokens <= 0 || D <= 0 || D > 12288 || top <= 0) return PG_ERR_ARG;
+  cudaStream_t st = PG_ST(stream);
+  const bool vec = D % 4 == 0 && ldy % 4 == 0 && ((reinterpret_cast<uintptr_t>(expert_out) | reinterpret_cast<uintptr_t>(norm_w) | reinterpret_cast<uintptr_t>(x) |
+                                                   reinterpret_cast<uintptr_t>(out_act)) & 15) == 0;
+  const size_t smem = (size_t)D * sizeof(float);
+#define PG_CN(TA, VEC) moe_combine_norm_add_kernel<TA, VEC><<<tokens, 256, smem, st>>>(expert_out, ldy, pair_row, weights, norm_w, x, static_cast<TA*>(out_act), D, top, eps)
+  if (act_f32) { if (vec) PG_CN(float, true); else PG_CN(float, false); }
+  else { if (vec) PG_CN(bf16, true); else PG_CN(bf16, false); }
+#undef PG_CN
+  PG_RET();
+}
+
 extern "C" int pg_moe_route(const float* logits, long long ld, const float* correction, int* ids, float* weights, int* counts, int tokens, int n_all,
-                            int n_real, int top, int group_count, int group_keep, float scale, const float* logit_bias, void* stream) {
+                            int n_real, int top, int group_count, int group_keep, float scale, const float* logit_bias, int flags, void* stream) {
   if (tokens <= 0 || n_all <= 0 || n_real < 0 || n_real > n_all || top <= 0 || top > n_all) return PG_ERR_ARG;
   if (group_count > 1 && (n_all % group_count != 0 || group_keep <= 0 || group_keep > group_count || group_count > 256)) return PG_ERR_ARG;
   if (group_count > 1 && top > (long long)group_keep * (n_all / group_count)) return PG_ERR_ARG;
@@ -444,7 +538,7 @@ extern "C" int pg_moe_route(const float* logits, long long ld, const float* corr
   cudaStream_t st = PG_ST(stream);
   if (n_real > 0 && cudaMemsetAsync(counts, 0, (size_t)n_real * sizeof(int), st) != cudaSuccess) return PG_ERR_CUDA;
   moe_route_kernel<<<(tokens + 3) / 4, 128, smem, st>>>(logits, ld, correction, ids, weights, counts, tokens, n_all, n_real, top, group_count, group_keep,
-                                                        scale, logit_bias);
+                                                        scale, logit_bias, flags);
   PG_RET();
 }
 
@@ -505,7 +599,7 @@ extern "C" int pg_moe_gather_rows(const void* x, long long ldx, const int* sorte
 }
 
 // Every expert's run of gathered rows through two dense tensor-core products (tcgen05 kernels of pg_gemm_bf16), issued from
-// here so that a layer costs one call from the host: mid = relu(xg W_up^T)^2 (bf16), eo = mid W_down^T (fp32).  One run is a few
+// here so that a layer costs one call from the host: mid = act(xg W_up^T) (bf16), eo = mid W_down^T (fp32).  One run is a few
 // dozen output tiles -- a fraction of the SMs -- so the experts are spread over four side streams that fork from and join the
 // caller's stream (the two products of one expert stay in order on one of them).
 namespace {
@@ -533,8 +627,9 @@ SideStreams* side_streams() {
 }  // namespace
 
 extern "C" int pg_moe_dense_runs(const void* xg, long long ldx, const void* w_up, const void* w_down, void* mid, long long ldm, float* eo, long long ldo,
-                                 const int* counts_host, int n_real, int D, int F, int glu, void* stream) {
-  if (n_real <= 0 || D <= 0 || F <= 0 || counts_host == nullptr || (glu && (F % 64) != 0)) return PG_ERR_ARG;
+                                 const int* counts_host, int n_real, int D, int F, int act, void* stream) {
+  const bool glu = act == 3;
+  if (n_real <= 0 || D <= 0 || F <= 0 || counts_host == nullptr || (glu && (F % 64) != 0) || (act != 2 && act != 3 && act != 6)) return PG_ERR_ARG;
   const int up_rows = glu ? 2 * F : F;  // gated experts: [64 gate | 64 up] packed rows, the gated unit in the product's epilogue
   const bf16* x = static_cast<const bf16*>(xg);
   const bf16* wu = static_cast<const bf16*>(w_up);
@@ -557,7 +652,7 @@ extern "C" int pg_moe_dense_runs(const void* xg, long long ldx, const void* w_up
     void* st = ss != nullptr ? static_cast<void*>(ss->s[used++ % kSideStreams]) : stream;
     const int swap = c <= 128 ? 1 : 0;
     rc = pg_gemm_bf16(x + off * ldx, ldx, wu + (long long)e * up_rows * D, D, m + off * ldm, ldm, nullptr, nullptr, 0, c, up_rows, D,
-                      glu ? PG_EPI_GEGLU : PG_EPI_BF16, glu ? 3 : 2, 1.0f, swap, 1, st);
+                      glu ? PG_EPI_GEGLU : PG_EPI_BF16, act, 1.0f, swap, 1, st);
     if (rc == PG_OK)
       rc = pg_gemm_bf16(m + off * ldm, ldm, wd + (long long)e * D * F, F, eo + off * ldo, ldo, nullptr, nullptr, 0, c, D, F, PG_EPI_F32, 0, 1.0f, swap, 1, st);
     off += c;

@@ -609,12 +609,13 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(const float* __res
       float v[V], z[V], ww[V];
       ldv<V>(o, t * D + base + d, v);
       if (gate_mode != 0) ldv<V>(gate, t * ldg + base + d, z);
-      ldv<V>(w, w_n == gs ? d : base + d, ww);
+      if (w != nullptr) ldv<V>(w, w_n == gs ? d : base + d, ww);
 #pragma unroll
       for (int i = 0; i < V; ++i) {
         if (gate_mode == 2) v[i] *= silu(z[i]);
-        v[i] *= iv * ww[i];
+        v[i] *= w != nullptr ? iv * ww[i] : iv;
         if (gate_mode == 1) v[i] *= sigmoid(z[i]);
+        if (gate_mode == 3) v[i] *= silu(z[i]);
       }
       stv<V>(out, t * ldo + base + d, v);
     }
@@ -653,7 +654,7 @@ __global__ void __launch_bounds__(256) group_norm_gate_flat_kernel(const float* 
       if (gate_mode != 0) {
         const float sg = sizeof(TA) == 2 ? fast_sigmoid(z[i][k]) : sigmoid(z[i][k]);
         if (gate_mode == 2) v[i][k] *= z[i][k] * sg;
-        z[i][k] = sg;
+        z[i][k] = gate_mode == 3 ? z[i][k] * sg : sg;
       }
       s = fmaf(v[i][k], v[i][k], s);
     }
@@ -664,9 +665,9 @@ __global__ void __launch_bounds__(256) group_norm_gate_flat_kernel(const float* 
   for (int i = 0; i < NV; ++i) {
     const int in = (i * lanes + l) * 4;
     float ww[4];
-    ldv<4>(w, w_n == gs ? in : col0 + in, ww);
+    if (w != nullptr) ldv<4>(w, w_n == gs ? in : col0 + in, ww);
 #pragma unroll
-    for (int k = 0; k < 4; ++k) v[i][k] *= iv * ww[k] * (gate_mode == 1 ? z[i][k] : 1.0f);
+    for (int k = 0; k < 4; ++k) v[i][k] *= (w != nullptr ? iv * ww[k] : iv) * ((gate_mode & 1) ? z[i][k] : 1.0f);
     stv<4>(out, t * ldo + col0 + in, v[i]);
   }
 }
@@ -837,7 +838,7 @@ extern "C" int pg_gated_scan(const PgGatedArgs* a, int kind, int n_min, int n_ma
 
 extern "C" int pg_group_norm_gate(const float* o, const float* w, int w_n, const void* gate, long long ldg, int gate_mode, void* out, long long ldo,
                                   int rows, int D, int groups, float eps, float scale, int act_f32, void* stream) {
-  if (rows <= 0 || D <= 0 || groups <= 0 || D % groups || (w_n != D && w_n != D / groups) || gate_mode < 0 || gate_mode > 2 || (gate_mode && gate == nullptr))
+  if (rows <= 0 || D <= 0 || groups <= 0 || D % groups || (w != nullptr && w_n != D && w_n != D / groups) || gate_mode < 0 || gate_mode > 3 || (gate_mode && gate == nullptr))
     return PG_ERR_ARG;
   const int gs = D / groups, ab = act_f32 ? 4 : 2;
   auto fits = [&](int v) {

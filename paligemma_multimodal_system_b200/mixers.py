@@ -5,9 +5,10 @@
                           sigmoid output gate
   LightningAttention      decayed linear attention with a per-sequence fp32 state, gated RMS norm over the joined heads
   WindowedSoftmaxAttention grouped-query softmax attention over a sliding window of the paged cache; optional, each a parameter:
-                          projection biases, weightless q/k RMS norm, partial interleaved rotation, a logarithmic distance penalty,
-                          a per-head score multiplier, a softmax sink, kept first keys, a per-head sigmoid output gate, keys and
-                          values borrowed from an earlier layer's cache
+                          projection biases, weightless q/k RMS norm per head or a weighted one over the whole projection, partial
+                          interleaved rotation with ramped frequencies, a logarithmic distance penalty, a per-head score
+                          multiplier, a softmax sink, kept first keys, a per-head sigmoid output gate, keys and values borrowed from
+                          an earlier layer's cache, values blended with an earlier layer's
   GegluFeedForward        W_down(gelu_tanh(W_gate h) * W_up h)
   GluFeedForward          W_down(act(W_gate h) * W_up h) with act = silu or relu, or the clamped form min(g, c) sigmoid(a min(g, c)) (clamp(u) + 1);
                           optional biases
@@ -19,6 +20,7 @@
   ProjectedMixer          base of the sub-layers below: one input projection for everything read from h (and, on request, for rows the caller
                           adds), a core that maps its columns to the activations of one output projection
   LogisticAttention       grouped-query attention whose weights are sigmoid(score + bias), not normalised over the keys; half-split rotation
+  Retention               fixed-decay linear attention with rotated queries and keys; per-head output norm without a weight, silu gate
   ChannelDeltaRule        gated delta rule with one decay per head and key channel behind short convolutions; per-head output norm and gate
   StateSpaceMixer         scalar-decay state-space recurrence (Mamba-2) behind a short convolution; gate before a grouped output norm
   MatrixMemory            matrix memory with exponential gates, running maximum and normaliser (mLSTM); per-head output norm and gate
@@ -124,11 +126,15 @@ class WindowedSoftmaxAttention:
     them, after its norm and rotation) with its own queries, window and score.
 
     value_is_key: there is no value projection; the values are the keys as projected, before norm and rotation (vdim == dim).
-    unit_sink: the softmax denominator is enlarged by exactly one (a sink whose logit is 0, no tensor)."""
+    unit_sink: the softmax denominator is enlarged by exactly one (a sink whose logit is 0, no tensor).
+    qk_norm "projection": RMS norms over all of q and all of k at once, before the split into heads, with weights (tensors q.norm, k.norm).
+    rot_scaling = dict(factor, original, fast, slow): ramped frequency rescaling with its cos / sin gain (ramped_rotary_frequencies).
+    value_blend "first": the layer's values are left for later layers of the step; "later": v <- (1 - l) v + l v_first of the same token, l the
+    tensor vmix (which a "first" layer carries unused); the blended values are what is cached."""
 
     def __init__(self, width, heads, kv_heads, dim, vdim, scale, eps, window=None, keep_first=0, bias=False, qk_norm=False, rot_dims=0,
                  rot_base=10000.0, distance_penalty=False, temperature=False, sink=False, head_gate=False, kv_from=None, value_is_key=False,
-                 unit_sink=False):
+                 unit_sink=False, rot_scaling=None, value_blend=None):
         if heads % kv_heads:
             raise ValueError("query heads must be a multiple of key/value heads")
         if rot_dims % 2 or rot_dims > dim:
@@ -137,7 +143,7 @@ class WindowedSoftmaxAttention:
             raise ValueError("a window holds at least the token itself")
         self.D, self.H, self.G, self.dim, self.vdim = int(width), int(heads), int(kv_heads), int(dim), int(vdim)
         self.scale, self.eps, self.window, self.keep_first = float(scale), float(eps), (int(window) if window is not None else None), int(keep_first)
-        self.bias, self.qk_norm, self.rot_dims = bool(bias), bool(qk_norm), int(rot_dims)
+        self.bias, self.qk_norm, self.rot_dims = bool(bias), (seq_ops.NORM_PROJECTION if qk_norm == "projection" else bool(qk_norm)), int(rot_dims)
         self.distance_penalty, self.temperature, self.sink, self.head_gate = bool(distance_penalty), bool(temperature), bool(sink), bool(head_gate)
         self.kv_from = None if kv_from is None else int(kv_from)
         self.value_is_key, self.unit_sink = bool(value_is_key), bool(unit_sink)
@@ -145,10 +151,19 @@ class WindowedSoftmaxAttention:
             raise ValueError("values that are the keys have the keys' size")
         if self.unit_sink and self.sink:
             raise ValueError("a layer has a learned sink or the unit one, not both")
-        self.freq = rotary_frequencies(rot_base, rot_dims) if rot_dims else torch.zeros(1, dtype=torch.float64)
+        if value_blend not in (None, "first", "later") or (value_blend and (self.value_is_key or self.kv_from is not None)):
+            raise ValueError("value_blend is None, 'first' or 'later', on a layer with value projections of its own")
+        self.value_blend, self.rot_gain = value_blend, 1.0
+        if rot_dims and rot_scaling:
+            self.freq, self.rot_gain = ramped_rotary_frequencies(rot_base, rot_dims, *(rot_scaling[k] for k in ("factor", "original", "fast", "slow")))
+        else:
+            self.freq = rotary_frequencies(rot_base, rot_dims) if rot_dims else torch.zeros(1, dtype=torch.float64)
 
     def cache_spec(self):
         return None if self.kv_from is not None else ("kv", self.G * self.dim, self.G * self.vdim)
+
+    def cache_specs(self):
+        return [self.cache_spec()]
 
     def load(self, take, pre):
         H, G, dim, vdim, D = self.H, self.G, self.dim, self.vdim, self.D
@@ -163,6 +178,12 @@ class WindowedSoftmaxAttention:
                 w["kb"] = take(pre + "k.b", (G * dim,))
                 if not self.value_is_key:
                     w["vb"] = take(pre + "v.b", (G * vdim,))
+        if self.qk_norm is seq_ops.NORM_PROJECTION:
+            w["qn"] = take(pre + "q.norm", (H * dim,))
+            if self.kv_from is None:
+                w["kn"] = take(pre + "k.norm", (G * dim,))
+        if self.value_blend:
+            w["vmix"] = take(pre + "vmix", ())
         if self.distance_penalty:
             w["r1"], w["r2"] = take(pre + "r1", (H,)), take(pre + "r2", (H,))
         if self.temperature:
@@ -195,6 +216,8 @@ class WindowedSoftmaxAttention:
         def vec(name):
             return w[name].to(**f32).contiguous() if name in w else None
 
+        self.qn, self.kn = vec("qn"), vec("kn")
+        self.v_mix = float(w["vmix"]) if self.value_blend == "later" else 0.0
         sink = torch.zeros(H, **f32) if self.unit_sink else vec("sink")  # exp(0) = 1 joins the denominator
         self.score = seq_ops.ScoreOptions(H, self.window, self.keep_first, sink=sink, dist_a=vec("r1"), dist_b=vec("r2"), head_scale=vec("temp"))
 
@@ -205,8 +228,13 @@ class WindowedSoftmaxAttention:
         own = self.kv_from is None
         src = li if own else self.kv_from
         kp, vp = store.k_pages[src], store.v_pages[src]
-        seq_ops.attn_prepare(proj, b, self.freq_d, None, None, q, kp if own else None, vp if own else None, H, G, dim, vdim, self.rot_dims, self.eps,
-                             PAGE, norm_qk=self.qk_norm, norm_v=False, v_from_k=self.value_is_key)
+        other = None
+        if self.value_blend == "first":
+            b.shared["values"] = proj[:, (H + G) * dim:(H + G) * dim + G * vdim]
+        elif self.value_blend == "later":
+            other = b.shared["values"]
+        seq_ops.attn_prepare(proj, b, self.freq_d, self.qn, self.kn, q, kp if own else None, vp if own else None, H, G, dim, vdim, self.rot_dims, self.eps,
+                             PAGE, norm_qk=self.qk_norm, norm_v=False, v_from_k=self.value_is_key, rot_gain=self.rot_gain, v_other=other, v_mix=self.v_mix)
         att = prec.empty(b.T, H * vdim)
         gate = proj[:, self.gate_col:] if self.head_gate else None
         seq_ops.attn_ragged(q, kp, vp, gate, att, b, H, G, dim, vdim, self.scale, 0.0, PAGE, gate_per_head=True, score=self.score)
@@ -547,18 +575,29 @@ class RoutedFeedForward:
     """Mixture of experts.  Router: p = softmax(W_r h + b_r) in fp32 over `experts + identity` outputs; the choice uses
     p + correction, limited to the `group_keep` best of `group_count` runs of neighbouring outputs; the `top` chosen outputs
     weigh in with p / sum(p chosen) * scale (without a correction that is the softmax over the chosen logits alone, chosen by
-    the largest logits).  The last `identity` outputs return h itself.  A shared expert (optional) is added for every token,
-    times sigmoid(w_sg . h) when it is gated.  activation "relu2": experts W_down relu(W_up h)^2; "silu_glu": experts
-    W_down (silu(W_gate h) * W_up h)."""
+    the largest logits).  scores "logistic": p = sigmoid(z) instead of the softmax; group_best 2: a group counts the sum of its two best
+    choices instead of the best; normalize False: the weights are p * scale.  The last `identity` outputs return h itself.  A shared expert (optional) is added for every token,
+    times sigmoid(w_sg . h) when it is gated.  activation "relu2": experts W_down relu(W_up h)^2; "gelu": experts
+    W_down gelu(W_up h), the erf form; "silu_glu": experts W_down (silu(W_gate h) * W_up h)."""
 
     def __init__(self, width, experts, identity, top, group_count, group_keep, scale, expert_ff, shared_ff, activation="relu2",
-                 correction=True, router_bias=False, shared_gate=False):
-        if activation not in ("relu2", "silu_glu"):
+                 correction=True, router_bias=False, shared_gate=False, scores="softmax", group_best=1, normalize=True):
+        acts = {"relu2": seq_ops.ACT_RELU2, "silu_glu": seq_ops.ACT_SILU_GLU, "gelu": seq_ops.ACT_GELU_ERF}
+        if activation not in acts:
             raise ValueError(f"unknown expert activation {activation!r}")
+        if scores not in ("softmax", "logistic") or group_best not in (1, 2):
+            raise ValueError("scores are 'softmax' or 'logistic', a group counts its best one or two choices")
+        if shared_ff and activation == "gelu":
+            raise ValueError("no shared expert with this activation")
+        self.act = acts[activation]
+        self.route_flags = ((seq_ops.ROUTE_LOGISTIC if scores == "logistic" else 0) | (seq_ops.ROUTE_GROUP_BEST_TWO if group_best == 2 else 0)
+                            | (0 if normalize else seq_ops.ROUTE_PLAIN_WEIGHTS))
         self.D, self.n_real, self.n_all, self.top = width, int(experts), int(experts) + int(identity), int(top)
         self.group_count, self.group_keep, self.scale, self.F = int(group_count), int(group_keep), float(scale), int(expert_ff)
         if self.group_count > 1 and self.n_all % self.group_count:
             raise ValueError("router outputs must divide into equal groups")
+        if not 1 <= self.top <= (self.n_all if self.group_count <= 1 else self.group_keep * (self.n_all // self.group_count)):
+            raise ValueError("more choices than eligible router outputs")
         self.glu, self.has_correction, self.router_bias = activation == "silu_glu", bool(correction), bool(router_bias)
         if not shared_ff:
             self.shared = None
@@ -628,19 +667,32 @@ class RoutedFeedForward:
             eo = torch.empty(plan.pairs, self.D, device="cuda", dtype=torch.float32)
             w_up = self.w_up_dense if self.glu else self.w_up
             _lib.check(_lib.lib().pg_moe_dense_runs(xg.data_ptr(), xg.stride(0), w_up.data_ptr(), self.w_down.data_ptr(), mid.data_ptr(), mid.stride(0),
-                                                    eo.data_ptr(), eo.stride(0), C.addressof(per), self.n_real, self.D, self.F, int(self.glu), _lib.stream()),
+                                                    eo.data_ptr(), eo.stride(0), C.addressof(per), self.n_real, self.D, self.F, self.act, _lib.stream()),
                        "pg_moe_dense_runs")
             return eo
-        mid = seq_ops.moe_gemm(h, plan, self.w_up, prec.empty(plan.pairs, self.F), gather=True, act=seq_ops.ACT_SILU_GLU if self.glu else seq_ops.ACT_RELU2)
+        mid = seq_ops.moe_gemm(h, plan, self.w_up, prec.empty(plan.pairs, self.F), gather=True, act=self.act)
         return seq_ops.moe_gemm(mid, plan, self.w_down, torch.empty(plan.pairs, self.D, device="cuda", dtype=torch.float32), gather=False)
 
-    def __call__(self, h, b, prec, resid=None):
+    def _routed(self, h, prec):
+        """Router logits, choice and expert rows of the step."""
         T = h.shape[0]
         z = seq_ops.linear(h, self.w_router, torch.empty(T, self.w_router.shape[0], device="cuda", dtype=torch.float32))
         ids, wts, counts = seq_ops.moe_route(z[:, :self.n_all], self.correction, self.n_real, self.top, self.group_count, self.group_keep, self.scale,
-                                             logit_bias=self.router_b)
+                                             logit_bias=self.router_b, flags=self.route_flags)
         plan = seq_ops.MoePlan(ids, counts, max(1, self.n_real))
-        eo = self.expert_products(h, plan, counts, prec) if self.n_real else None
+        return z, ids, wts, plan, self.expert_products(h, plan, counts, prec) if self.n_real else None
+
+    def add_normed(self, h, prec, norm_w, x, out_act, eps):
+        """x += N(experts(h)) * norm_w in place (RMS norm), out_act a copy of the new rows: combine, norm and residual in one pass.  For layers
+        without identity outputs and without a shared expert."""
+        if self.shared is not None or self.n_real != self.n_all:
+            raise ValueError("identity outputs and shared experts are not part of the fused combine")
+        _, _, wts, plan, eo = self._routed(h, prec)
+        seq_ops.moe_combine_norm_add(eo, plan, wts, norm_w, x, out_act, eps)
+
+    def __call__(self, h, b, prec, resid=None):
+        T = h.shape[0]
+        z, ids, wts, plan, eo = self._routed(h, prec)
         sh = self.shared(h, b, prec) if self.shared is not None else None
         sg = z[:, self.n_all:self.n_all + 1] if self.shared_gate else None
         if resid is not None:
@@ -929,6 +981,62 @@ class MatrixMemory(ProjectedMixer):
         seq_ops.gated_recurrence(seq_ops.MATRIX_MEMORY, cols["q"], cols["k"], cols["v"], cols["i"], cols["f"], self.ib, self.fb, None, store.state[li],
                                  store.state[li + 1], o, b, H, H, dim, vdim, qscale=dim ** -0.5, cap=self.cap)
         seq_ops.group_norm_gate(o, self.norm, cols["g"], out, H, self.eps, seq_ops.GATE_SIGMOID_AFTER, self.out_scale)
+
+
+class Retention(ProjectedMixer):
+    """q = W_q h, k = W_k h, v = W_v h; q and k rotated (first rot_dims dimensions of every head), k times dim^-1/2; per head with a fixed decay
+        S <- decay S + k v^T;  o = S^T q;  out = o / rms(o) * silu(W_g h)      (norm per head, no weight).
+    rot_layout "half" pairs element i with i + rot_dims / 2 (the rows of W_q and W_k are reordered once so that partners are neighbours: dot
+    products and the state's read-out do not change), "interleaved" 2i with 2i + 1."""
+
+    def __init__(self, width, heads, dim, vdim, decay, eps, rot_dims=0, rot_base=10000.0, rot_layout="half"):
+        if len(decay) != int(heads):
+            raise ValueError("one decay per head")
+        if rot_dims % 2 or rot_dims > dim:
+            raise ValueError("rotary dimensions must be even and at most the head size")
+        if rot_layout not in ("half", "interleaved"):
+            raise ValueError("rot_layout is 'half' or 'interleaved'")
+        self.D, self.H, self.dim, self.vdim, self.eps = int(width), int(heads), int(dim), int(vdim), float(eps)
+        self.inner, self.rot_dims, self.rot_base, self.rot_layout = self.H * self.vdim, int(rot_dims), float(rot_base), rot_layout
+        self.decay = torch.tensor([float(a) for a in decay], dtype=torch.float32)
+        self.freq = rotary_frequencies(rot_base, rot_dims) if rot_dims else torch.zeros(1, dtype=torch.float64)
+
+    def cache_specs(self):
+        return [("state", (self.H, self.dim, self.vdim))]
+
+    def load(self, take, pre):
+        H, dim, vdim, D = self.H, self.dim, self.vdim, self.D
+        self.w = dict(q=take(pre + "q", (H * dim, D)), k=take(pre + "k", (H * dim, D)), v=take(pre + "v", (H * vdim, D)), g=take(pre + "g", (H * vdim, D)),
+                      o=take(pre + "o", (D, H * vdim)))
+
+    def in_parts(self):
+        w = self.w
+        order = torch.tensor(half_to_pair_order(self.dim, self.rot_dims) if self.rot_layout == "half" else list(range(self.dim)))
+
+        def paired(t):
+            return t.view(self.H, self.dim, self.D)[:, order.to(t.device)].reshape(self.H * self.dim, self.D)
+
+        return {"qkv": torch.cat([paired(w["q"]), paired(w["k"]), w["v"]], 0), "g": w["g"]}
+
+    def out_weight(self):
+        return self.w["o"]
+
+    def pack_core(self, prec, pitch):
+        self.decay_d, self.freq_d = self.decay.to("cuda"), self.freq.to("cuda")
+
+    def core(self, cols, b, store, li, prec, out):
+        H, dim, vdim = self.H, self.dim, self.vdim
+        turn = None
+        if self.rot_dims:  # one table per step for all layers that turn alike
+            key = ("rotary", self.rot_base, self.rot_dims, dim)
+            turn = b.shared.get(key) if b.shared is not None else None
+            if turn is None:
+                turn = seq_ops.rotary_table(b, self.freq_d, self.rot_dims, dim)
+                if b.shared is not None:
+                    b.shared[key] = turn
+        o = torch.empty(b.T, self.inner, device="cuda", dtype=torch.float32)
+        seq_ops.retention(cols["qkv"], store.state[li], self.decay_d, o, b, H, dim, vdim, kscale=dim ** -0.5, rotate=turn)
+        seq_ops.group_norm_gate(o, None, cols["g"], out, H, self.eps, seq_ops.GATE_SILU_AFTER, self.out_scale)
 
 
 class SideBySide(ProjectedMixer):

@@ -73,6 +73,11 @@ def _load_fadosun(path, dtype=torch.bfloat16, **kw):
     return load_fadosun(path, dtype)
 
 
+def _load_padulorn(path, dtype=torch.bfloat16, **kw):
+    from .modeling_padulorn import load_padulorn
+    return load_padulorn(path, dtype)
+
+
 for _n in ("paligemma", "PaliGemmaForConditionalGeneration"):
     register(_n, _load_paligemma)
 register("Mapedra", _load_mapedra)
@@ -80,3 +85,4 @@ register("Pukerax", _load_pukerax)
 register("Kovusun", _load_kovusun)
 register("Zigivik", _load_zigivik)
 register("Fadosun", _load_fadosun)
+register("Padulorn", _load_padulorn)

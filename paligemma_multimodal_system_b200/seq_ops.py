@@ -49,6 +49,9 @@ class StepBatch:
     dense_max_pages: int = 0
     dense_rows: int = 0       # rows of the scratch matrix (a multiple of the page size)
     dense_max_len: int = 0    # the longest ctx + n among those entries
+    # what one layer of the CURRENT step leaves for later ones (rotation tables, a layer's values); a model that uses it starts every step
+    # with a fresh one (`step_scope`)
+    shared: Optional[dict] = None
 
 
 def make_step_batch(entries: Sequence[dict]) -> StepBatch:
@@ -95,6 +98,11 @@ def make_step_batch(entries: Sequence[dict]) -> StepBatch:
                      dense_max_len=max(lens))
 
 
+def step_scope(b: StepBatch) -> StepBatch:
+    """The same step with an empty `shared`."""
+    return dataclasses.replace(b, shared={})
+
+
 class StaticDecodeBatch:
     """Fixed-address StepBatch for steps of E single-token entries (a decode step), so that the step can be captured once in a
     CUDA graph and replayed: `fill` rewrites the pinned host image and copies it over the device buffer in stream order.
@@ -132,7 +140,8 @@ def _aligned(t, n=16):
     return t.data_ptr() % n == 0
 
 
-ACT_NONE, ACT_GELU, ACT_RELU2, ACT_SILU_GLU = 0, 1, 2, 3  # ACT_SILU_GLU: grouped products only (gate / up rows alternate)
+# ACT_SILU_GLU: grouped products only (gate / up rows alternate); ACT_GELU is the tanh form, ACT_GELU_ERF the exact one
+ACT_NONE, ACT_GELU, ACT_RELU2, ACT_SILU_GLU, ACT_GELU_ERF = 0, 1, 2, 3, 6
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int = ACT_NONE, bias: Optional[torch.Tensor] = None):
@@ -257,9 +266,11 @@ def glu(gu, out, kind, limit=0.0, alpha=1.0):
     return out
 
 
-def embed_rows(tokens, table, col0, D, scale):
+def embed_rows(tokens, table, col0, D, scale, out_act=None):
+    """fp32 rows [tokens, D]; out_act (the table's type, [tokens, D]) receives a copy."""
     out = torch.empty(tokens.numel(), D, device="cuda", dtype=torch.float32)
-    _lib.check(_lib.lib().pg_embed_rows(tokens.data_ptr(), table.data_ptr(), table.stride(0), int(col0), out.data_ptr(), tokens.numel(), D,
+    assert out_act is None or (out_act.dtype == table.dtype and out_act.is_contiguous() and out_act.shape == out.shape)
+    _lib.check(_lib.lib().pg_embed_rows(tokens.data_ptr(), table.data_ptr(), table.stride(0), int(col0), out.data_ptr(), _lib.ptr(out_act), tokens.numel(), D,
                                         float(scale), int(table.dtype == torch.float32), _lib.stream()), "pg_embed_rows")
     return out
 
@@ -296,17 +307,25 @@ def side_gate(z, tokens, table, col0, out, n):
                                        out.stride(0), rows, int(n), n_pad, int(out.dtype == torch.float32), _lib.stream()), "pg_side_gate")
 
 
+NORM_PROJECTION = "projection"  # attn_prepare: one norm over all of q, one over all of k
+
+
 def attn_prepare(qkv, b: StepBatch, freq, q_norm, k_norm, q_out, k_pages, v_pages, H, G, dim, vdim, rot_dims, eps, page, norm_qk=True, norm_v=True,
-                 v_from_k=False):
+                 v_from_k=False, rot_gain=1.0, v_other=None, v_mix=0.0):
     """q_norm / k_norm None: norms without a weight; norm_qk / norm_v False: no q/k norm / no value norm; k_pages and v_pages None: the
     rows hold queries only (the layer attends over another layer's cache); v_from_k: the rows have no value columns, the values are the
-    keys as projected (before norm and rotation)."""
+    keys as projected (before norm and rotation); norm_qk NORM_PROJECTION: the norms run over all heads at once (weights of that size);
+    rot_gain multiplies cosines and sines; v_other [T, G * vdim]: the values become (1 - v_mix) v + v_mix v_other."""
+    for w, heads in ((q_norm, H), (k_norm, G)):
+        assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == (heads * dim if norm_qk is NORM_PROJECTION else dim))
+    assert v_other is None or (v_other.dtype == qkv.dtype and v_other.stride(1) == 1 and v_other.shape == (b.T, G * vdim))
     assert qkv.stride(1) == 1 and freq.dtype == torch.float64 and qkv.dtype == q_out.dtype and (k_pages is None) == (v_pages is None)
     assert k_pages is None or k_pages.dtype == qkv.dtype
     _lib.check(_lib.lib().pg_attn_prepare(qkv.data_ptr(), qkv.stride(0), b.pos.data_ptr(), b.row_entry.data_ptr(), b.page_table.data_ptr(),
                                           b.max_pages, page, freq.data_ptr(), _lib.ptr(q_norm), _lib.ptr(k_norm), q_out.data_ptr(),
-                                          _lib.ptr(k_pages), _lib.ptr(v_pages), b.T, H, G, dim, vdim, rot_dims, float(eps), int(bool(norm_qk)),
-                                          int(bool(norm_v)), int(bool(v_from_k)), int(qkv.dtype == torch.float32), _lib.stream()), "pg_attn_prepare")
+                                          _lib.ptr(k_pages), _lib.ptr(v_pages), b.T, H, G, dim, vdim, rot_dims, float(eps), 2 if norm_qk is NORM_PROJECTION else int(bool(norm_qk)),
+                                          int(bool(norm_v)), int(bool(v_from_k)), float(rot_gain), _lib.ptr(v_other), 0 if v_other is None else v_other.stride(0),
+                                          float(v_mix), int(qkv.dtype == torch.float32), _lib.stream()), "pg_attn_prepare")
 
 
 class ScoreOptions:
@@ -509,15 +528,20 @@ def dense_view(b: StepBatch) -> StepBatch:
 
 
 # ---- routed feed-forward ---------------------------------------------------------------------------------------------
-def moe_route(logits, correction, n_real, top, group_count, group_keep, scale, logit_bias=None):
-    """logits fp32 [T, n_all] (+ logit_bias fp32 [n_all]) -> ids int32 [T, top], weights fp32 [T, top], counts int32 [n_real] (device)."""
+ROUTE_LOGISTIC, ROUTE_GROUP_BEST_TWO, ROUTE_PLAIN_WEIGHTS = 1, 2, 4
+
+
+def moe_route(logits, correction, n_real, top, group_count, group_keep, scale, logit_bias=None, flags=0):
+    """logits fp32 [T, n_all] (+ logit_bias fp32 [n_all]) -> ids int32 [T, top], weights fp32 [T, top], counts int32 [n_real] (device).  flags:
+    ROUTE_LOGISTIC -- scores are sigmoid(logit) instead of the softmax; ROUTE_GROUP_BEST_TWO -- a group counts the sum of its two best
+    choices; ROUTE_PLAIN_WEIGHTS -- the chosen scores are not divided by their sum."""
     T, n_all = logits.shape
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     ids = torch.empty(T, top, device="cuda", dtype=torch.int32)
     wts = torch.empty(T, top, device="cuda", dtype=torch.float32)
     counts = torch.empty(max(1, n_real), device="cuda", dtype=torch.int32)
     _lib.check(_lib.lib().pg_moe_route(logits.data_ptr(), logits.stride(0), _lib.ptr(correction), ids.data_ptr(), wts.data_ptr(), counts.data_ptr(), T,
-                                       n_all, n_real, top, int(group_count), int(group_keep), float(scale), _lib.ptr(logit_bias), _lib.stream()), "pg_moe_route")
+                                       n_all, n_real, top, int(group_count), int(group_keep), float(scale), _lib.ptr(logit_bias), int(flags), _lib.stream()), "pg_moe_route")
     return ids, wts, counts
 
 
@@ -573,6 +597,16 @@ def moe_combine(expert_out, plan: MoePlan, ids, weights, h, shared_out, y, share
     return y
 
 
+def moe_combine_norm_add(expert_out, plan: MoePlan, weights, norm_w, x, out_act, eps):
+    """y = sum_k weights[t, k] * expert row; x += y / rms(y) * norm_w in place; out_act (may be None) gets the new row."""
+    T, D = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and expert_out.dtype == torch.float32 and expert_out.stride(1) == 1 and norm_w.numel() == D
+    assert norm_w.dtype == torch.float32 and (out_act is None or (out_act.is_contiguous() and out_act.shape == x.shape))
+    _lib.check(_lib.lib().pg_moe_combine_norm_add(expert_out.data_ptr(), expert_out.stride(0), plan.pair_row.data_ptr(), weights.data_ptr(), norm_w.data_ptr(),
+                                                  x.data_ptr(), _lib.ptr(out_act), T, D, plan.top, float(eps),
+                                                  int(out_act is not None and out_act.dtype == torch.float32), _lib.stream()), "pg_moe_combine_norm_add")
+
+
 # a portion at least this long is advanced in 32-token blocks; shorter ones (decode above all) token by token
 LINEAR_ATTN_CHUNK_MIN = 8
 
@@ -583,7 +617,43 @@ def linear_attn(qkv, state, decay, out, b: StepBatch, H, dim, vdim, chunked=None
         chunked = b.max_n >= LINEAR_ATTN_CHUNK_MIN
     fn = _lib.lib().pg_linear_attn_chunked if chunked else _lib.lib().pg_linear_attn_scan
     _lib.check(fn(qkv.data_ptr(), qkv.stride(0), state.data_ptr(), decay.data_ptr(), out.data_ptr(), b.row0.data_ptr(), b.n.data_ptr(),
-                  b.ctx.data_ptr(), b.slot.data_ptr(), b.E, H, dim, vdim, int(qkv.dtype == torch.float32), _lib.stream()), "pg_linear_attn")
+                  b.ctx.data_ptr(), b.slot.data_ptr(), b.E, H, dim, vdim, 0, int(qkv.dtype == torch.float32), _lib.stream()), "pg_linear_attn")
+
+
+def rotary_table(b: StepBatch, freq, rot_dims, dim, gain=1.0):
+    """fp32 [T, 2, pairs]: cosines and sines of the step's rows for every pair of a head of `dim` elements (1 and 0 past the rotated ones)."""
+    pairs = (dim + 7) // 8 * 4
+    assert freq.dtype == torch.float64 and rot_dims <= dim
+    out = torch.empty(b.T, 2, pairs, device="cuda", dtype=torch.float32)
+    _lib.check(_lib.lib().pg_rotary_table(b.pos.data_ptr(), freq.data_ptr(), out.data_ptr(), b.T, int(rot_dims), pairs, float(gain), _lib.stream()), "pg_rotary_table")
+    return out
+
+
+def retention(qkv, state, decay, out, b: StepBatch, H, dim, vdim, kscale=1.0, rotate=None, blocks=None):
+    """S <- decay S + k v^T, out = S^T q per head (fp32 [T, H * vdim]) with q and k turned in neighbouring pairs by `rotate` (rotary_table; None:
+    not turned) and k times kscale.  Entries with several new tokens go in blocks -- on the tensor cores for bf16 head sizes that fit --
+    the others token by token (blocks True / False: one form for every entry); an entry's own length decides."""
+    import ctypes as C
+    assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, dim, vdim) and out.dtype == torch.float32 and out.is_contiguous() and qkv.stride(1) == 1
+    assert rotate is None or (rotate.dtype == torch.float32 and rotate.is_contiguous() and rotate.shape[0] == b.T and 2 * rotate.shape[2] >= dim)
+    f32 = int(qkv.dtype == torch.float32)
+    tensor_cores = not f32 and dim % 8 == 0 and dim <= 128 and vdim % 8 == 0 and qkv.stride(0) % 8 == 0 and _aligned(qkv)
+    n_min = {None: RECURRENCE_BLOCK_MIN if tensor_cores else LINEAR_ATTN_CHUNK_MIN, True: 1, False: FOREVER}[blocks]
+
+    def go(fn, lo, hi, *tail):
+        ops = _lib.LinearAttnOps(0, float(kscale), _lib.ptr(rotate), 0 if rotate is None else rotate.shape[2], lo, hi)
+        _lib.check(fn(qkv.data_ptr(), qkv.stride(0), state.data_ptr(), decay.data_ptr(), out.data_ptr(), b.row0.data_ptr(), b.n.data_ptr(), b.ctx.data_ptr(),
+                      b.slot.data_ptr(), b.E, H, dim, vdim, C.addressof(ops), *tail, _lib.stream()), "pg_linear_attn")
+
+    L = _lib.lib()
+    if b.max_n >= n_min:
+        if tensor_cores:
+            go(L.pg_linear_attn_blocks, n_min, FOREVER)
+        else:
+            go(L.pg_linear_attn_chunked, n_min, FOREVER, f32)
+    if b.max_n < n_min or (n_min > 1 and b.E > 1):
+        go(L.pg_linear_attn_scan, 1, n_min - 1, f32)
+    return out
 
 
 # ---- recurrent mixers --------------------------------------------------------------------------------------------------
@@ -689,16 +759,17 @@ def gated_recurrence(kind, q, k, v, gate1, gate2, p1, p2, p3, state, norm_state,
     return out
 
 
-GATE_NONE, GATE_SIGMOID_AFTER, GATE_SILU_BEFORE = 0, 1, 2
+GATE_NONE, GATE_SIGMOID_AFTER, GATE_SILU_BEFORE, GATE_SILU_AFTER = 0, 1, 2, 3
 
 
 def group_norm_gate(o, w, gate, out, groups, eps, mode, scale=1.0):
-    """out = scale * norm(o) * w * sigmoid(gate) (GATE_SIGMOID_AFTER) or scale * norm(o * silu(gate)) * w (GATE_SILU_BEFORE), the norm in `groups`
-    equal parts of the row; w fp32 [D] or one group's [D / groups]; out may be a column slice."""
+    """out = scale * norm(o) * w * sigmoid(gate) (GATE_SIGMOID_AFTER), * silu(gate) (GATE_SILU_AFTER) or scale * norm(o * silu(gate)) * w
+    (GATE_SILU_BEFORE), the norm in `groups` equal parts of the row; w fp32 [D], one group's [D / groups] or None; out may be a column slice."""
     rows, D = o.shape
-    assert o.dtype == torch.float32 and o.is_contiguous() and w.dtype == torch.float32 and w.is_contiguous() and out.shape == o.shape and out.stride(1) == 1
+    assert o.dtype == torch.float32 and o.is_contiguous() and out.shape == o.shape and out.stride(1) == 1
+    assert w is None or (w.dtype == torch.float32 and w.is_contiguous())
     assert gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1)
-    _lib.check(_lib.lib().pg_group_norm_gate(o.data_ptr(), w.data_ptr(), w.numel(), _lib.ptr(gate), 0 if gate is None else gate.stride(0), int(mode),
+    _lib.check(_lib.lib().pg_group_norm_gate(o.data_ptr(), _lib.ptr(w), 0 if w is None else w.numel(), _lib.ptr(gate), 0 if gate is None else gate.stride(0), int(mode),
                                              out.data_ptr(), out.stride(0), rows, D, int(groups), float(eps), float(scale), int(out.dtype == torch.float32),
                                              _lib.stream()), "pg_group_norm_gate")
     return out
