@@ -1029,3 +1029,194 @@ def run_fadosun(args):
             out[key] = round(out[key], 1)
     print(json.dumps(out), flush=True)
     return out
+
+
+# ----------------------------------------------------------------------------------------------------------------------
+# `bench.py --arch padulorn`: the Padulorn decoder beside the Mapedra decoder (the closest model of the package: norms on the sub-layer outputs,
+# three layers of decayed linear attention to one of softmax attention) at equal width / heads / k/v heads / head size / depth, and its
+# routed experts beside the routed feed-forward of the Pukerax decoder at equal sizes
+# ----------------------------------------------------------------------------------------------------------------------
+def padulorn_config(width, heads, kv_heads, dim, ff, vocab, layers, every=4, experts=16, top=4):
+    """`every`-th layer attention (window 1024, 16 kept tokens), the others retention; on every layer 16 experts of width ff / 8, top 4, four
+    groups of which two are kept."""
+    mlp = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "v_mix": True, "mask": {"size": 1024, "keep_first": 16},
+           "rot": {"base": 1e6, "dims": dim // 2, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    ret = {"heads": heads, "dim": dim, "vdim": dim, "decay": [1.0 - 2.0 ** (-5 - 5 * h / heads) for h in range(heads)], "rot": {"base": 1e6, "dims": dim}}
+    return {"architecture": "Padulorn", "vocab": vocab, "width": width, "embedding": {"scale": width ** 0.5}, "norm": {"eps": 1e-6}, "residual_mult": 0.6,
+            "logit_scale": 0.5, "layers": [dict({"type": "attention", "mixer": att} if (i + 1) % every == 0 else {"type": "retention", "mixer": ret}, mlp=mlp)
+                                           for i in range(layers)]}
+
+
+def random_padulorn(cfg, seed=0):
+    from .modeling_padulorn import PadulornConfig, PadulornForCausalLM
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    c = PadulornConfig(cfg)
+    model = PadulornForCausalLM(c, torch.bfloat16)
+
+    def take(name, shape):
+        r = torch.randn(shape, device="cuda", generator=g)
+        t = 0.5 + 0.1 * r if not shape else 1.0 + 0.1 * r if len(shape) == 1 else r * shape[-1] ** -0.5
+        return t.to(torch.bfloat16)
+
+    model.embed = take("embed", (c.vocab, c.width))
+    for blk in model.blocks:
+        blk.load(take)
+    model.final_norm, model.head = take("final.norm", (c.width,)), take("head", (c.vocab, c.width))
+    model.pack()
+    return model
+
+
+def _routed_kernels(k, tag, ff, h, x, T, W, norm_w=None):
+    """Router, plan, expert products and combine of a routed feed-forward on T rows."""
+    prec = seq_ops.Precision(torch.bfloat16)
+    n, top, F = ff.n_real, ff.top, ff.F
+    z = seq_ops.linear(h, ff.w_router, torch.empty(T, ff.w_router.shape[0], device="cuda", dtype=torch.float32))
+
+    def route():
+        return seq_ops.moe_route(z[:, :ff.n_all], ff.correction, n, top, ff.group_count, ff.group_keep, ff.scale, logit_bias=ff.router_b, flags=ff.route_flags)
+
+    flush = _routed_kernels.flush
+    ids, wts, counts = route()
+    k[f"{tag}_route"] = dict(s=timed(route, flush=flush), bytes=T * (ff.n_all * 4 + top * 8))
+    k[f"{tag}_plan"] = dict(s=timed(lambda: seq_ops.MoePlan(ids, counts, n), flush=flush), bytes=T * top * 12)
+    plan = seq_ops.MoePlan(ids, counts, n)
+    used = int((counts > 0).sum())
+    k[f"{tag}_experts"] = dict(s=timed(lambda: ff.expert_products(h, plan, counts, prec), flush=flush), flops=4 * T * top * W * F,
+                               bytes=used * 2 * W * F * 2 + T * W * 2 + T * top * (F * 4 + W * 4))
+    eo = ff.expert_products(h, plan, counts, prec)
+    if norm_w is not None:
+        xa = prec.empty(T, W)
+        k[f"{tag}_combine_norm_residual"] = dict(s=timed(lambda: seq_ops.moe_combine_norm_add(eo, plan, wts, norm_w, x, xa, 1e-6), flush=flush),
+                                                 bytes=T * W * (top * 4 + 8 + 2))
+    else:
+        y = torch.empty(T, W, device="cuda", dtype=torch.float32)
+        k[f"{tag}_combine"] = dict(s=timed(lambda: seq_ops.moe_combine(eo, plan, ids, wts, h, None, y), flush=flush), bytes=T * W * (top * 4 + 4))
+
+
+def run_padulorn(args):
+    from .mixers import RoutedFeedForward
+    _lib.require_device()
+    torch.cuda.set_device(0)
+    hbm, tflops, src = peaks()
+    W, H, G, dh, F, V, L = args.width, args.heads, args.kv_heads, args.head_dim, args.ff, args.vocab, args.layers
+    B_pre, S, B_dec, ctx = args.prefill_batch, args.seq_len, args.decode_batch, args.context
+    flush = torch.zeros(64 * 1024 * 1024, device="cuda", dtype=torch.float32)  # 256 MB > L2
+    _routed_kernels.flush = flush
+    cfg = padulorn_config(W, H, G, dh, F, V, L)
+    out = {"metric": "padulorn_vs_mapedra_tokens_per_s", "dtype": "bf16", "data": "synthetic", "peaks": src,
+           "config": {"width": W, "heads": H, "kv_heads": G, "head_dim": dh, "experts": [16, F // 8, "top 4"], "mapedra_ff": F, "vocab": V, "layers": L,
+                      "prefill": [B_pre, S], "decode": [B_dec, ctx], "l2": "256 MB buffer rewritten before every timed launch"}}
+    model = random_padulorn(cfg)
+    eng = _throughput(model, args, flush, V, "padulorn", out)
+    prec, k, store = model.prec, {}, eng.store
+    inner = H * dh
+    li_att = next(i for i, l in enumerate(cfg["layers"]) if l["type"] == "attention")
+    li_ret = next(i for i, l in enumerate(cfg["layers"]) if l["type"] == "retention")
+    att, ret = model.blocks[li_att].mixer, model.blocks[li_ret].mixer
+    blk0 = model.blocks[0]
+    other_ff = RoutedFeedForward(W, 16, 0, 4, 4, 2, 2.5, F // 8, 0)  # the Pukerax form without identity outputs and shared expert
+    g = torch.Generator(device="cuda").manual_seed(3)
+    other_ff.load(lambda name, shape: (torch.randn(shape, device="cuda", generator=g) * shape[-1] ** -0.5).to(torch.bfloat16) * (0.01 if len(shape) == 1 else 1.0), "")
+    other_ff.pack(prec)
+    shapes = {"prefill": (B_pre, S, 0), "decode": (B_dec, 1, ctx)}
+    for name, (n_seq, n_new, c0) in shapes.items():
+        b = seq_ops.step_scope(_entries(store, n_seq, n_new, c0))
+        T = b.T
+        for t in store.state:
+            if t is not None:
+                t.normal_()
+        x, y = torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda")
+        h = torch.randn(T, W, device="cuda").to(torch.bfloat16)
+        xa = prec.empty(T, W)
+        k[f"norm_residual_{name}"] = dict(s=timed(lambda: seq_ops.group_rmsnorm_add(y, blk0.norm1_d, x, xa, 1, 1e-6), flush=flush), bytes=T * W * (4 + 8 + 2))
+        # retention
+        state_rw = n_seq * H * dh * dh * 4 * 2
+        proj = torch.randn(T, ret.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        cols = {n: proj[:, i:j] for n, (i, j) in ret.cols.items()}
+        turn = seq_ops.rotary_table(b, ret.freq_d, ret.rot_dims, dh)
+        o, mid = torch.empty(T, inner, device="cuda"), prec.empty(T, inner)
+        k[f"rotary_table_{name}"] = dict(s=timed(lambda: seq_ops.rotary_table(b, ret.freq_d, ret.rot_dims, dh), flush=flush), bytes=T * dh * 4)
+        k[f"retention_{name}"] = dict(
+            s=timed(lambda: seq_ops.retention(cols["qkv"], store.state[li_ret], ret.decay_d, o, b, H, dh, dh, kscale=dh ** -0.5, rotate=turn), flush=flush),
+            flops=T * H * 4 * dh * dh, bytes=state_rw + T * inner * (3 * 2 + 4))
+        k[f"head_norm_gate_{name}"] = dict(s=timed(lambda: seq_ops.group_norm_gate(o, None, cols["g"], mid, H, 1e-6, seq_ops.GATE_SILU_AFTER), flush=flush),
+                                           bytes=T * inner * (4 + 2 + 2))
+        # attention
+        proja = torch.randn(T, att.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        q, ao = prec.empty(T, inner), prec.empty(T, inner)
+        kp, vp = store.k_pages[li_att], store.v_pages[li_att]
+        kp.normal_()
+        vp.normal_()
+        vals = proja[:, (H + G) * dh:(H + 2 * G) * dh]
+        k[f"attn_prepare_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_prepare(proja, b, att.freq_d, att.qn, att.kn, q, kp, vp, H, G, dh, dh, att.rot_dims, 1e-6, PAGE, norm_qk=att.qk_norm,
+                                                 norm_v=False, rot_gain=att.rot_gain, v_other=vals, v_mix=0.3), flush=flush), bytes=T * ((H + 2 * G) * dh * 4 + G * dh * 2))
+        win = att.window or (c0 + n_new)
+        pairs = n_seq * sum(min(i + 1, win) + max(0, min(att.keep_first, i + 1 - win)) for i in range(c0, c0 + n_new))
+        k[f"attention_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_ragged(q, kp, vp, None, ao, b, H, G, dh, dh, att.scale, 0.0, PAGE, score=att.score), flush=flush),
+            flops=4 * dh * H * pairs, bytes=n_seq * min(c0 + n_new, win + att.keep_first + n_new) * G * 2 * dh * 2 + 2 * T * inner * 2)
+        k[f"mixer_retention_{name}"] = dict(
+            s=timed(lambda: ret(h, b, store, li_ret, prec), flush=flush), flops=2 * T * W * (ret.w_in.shape[0] + inner),
+            bytes=(ret.w_in.numel() + ret.w_o.numel()) * 2 + T * W * 6 + state_rw)
+        _routed_kernels(k, f"moe_{name}", blk0.ff, h, x, T, W, blk0.norm2_d)
+        _routed_kernels(k, f"pukerax_moe_{name}", other_ff, h, x, T, W)
+        for i in range(n_seq):
+            store.release(("k", i))
+    del eng, model, store
+    torch.cuda.empty_cache()
+
+    # ---------------------------------------------------------------- Mapedra at equal size
+    mm = random_mapedra(mapedra_config(W, H, G, dh, F, V, L))
+    eng = _throughput(mm, args, flush, V, "mapedra", out)
+    store, prec = eng.store, mm.prec
+    li_att = next(i for i, b in enumerate(mm.blocks) if hasattr(b.mixer, "G"))
+    li_lin = next(i for i, b in enumerate(mm.blocks) if hasattr(b.mixer, "decay"))
+    att, lin = mm.blocks[li_att].mixer, mm.blocks[li_lin].mixer
+    for name, (n_seq, n_new, c0) in shapes.items():
+        b = _entries(store, n_seq, n_new, c0)
+        T = b.T
+        proj = torch.randn(T, att.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        q, o = prec.empty(T, inner), prec.empty(T, inner)
+        kp, vp = store.k_pages[li_att], store.v_pages[li_att]
+        kp.normal_()
+        vp.normal_()
+        gate = proj[:, (H + G) * dh + G * dh:]
+        k[f"mapedra_attn_prepare_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_prepare(proj, b, att.freq_d, att.qn, att.kn, q, kp, vp, H, G, dh, dh, att.rot_dims, 1e-6, PAGE), flush=flush),
+            bytes=T * (H + 2 * G) * dh * 2 * 2)
+        pairs = n_seq * (n_new * c0 + n_new * (n_new + 1) // 2)
+        k[f"mapedra_attention_{name}"] = dict(
+            s=timed(lambda: seq_ops.attn_ragged(q, kp, vp, gate, o, b, H, G, dh, dh, att.scale, att.softcap, PAGE), flush=flush),
+            flops=4 * dh * H * pairs, bytes=n_seq * (c0 + n_new) * G * 2 * dh * 2 + 3 * T * inner * 2)
+        projl = torch.randn(T, lin.w_in.shape[0], device="cuda").to(torch.bfloat16)
+        ol = torch.empty(T, inner, device="cuda", dtype=torch.float32)
+        k[f"mapedra_lightning_{name}"] = dict(
+            s=timed(lambda: seq_ops.linear_attn(projl, store.state[li_lin], lin.decay_d, ol, b, H, dh, dh), flush=flush),
+            flops=T * H * 4 * dh * dh, bytes=n_seq * H * dh * dh * 4 * 2 + T * inner * (3 * 2 + 4))
+        attl = prec.empty(T, inner)
+        k[f"mapedra_lightning_norm_gate_{name}"] = dict(
+            s=timed(lambda: seq_ops.rmsnorm_gate(ol, lin.norm, projl[:, 3 * inner:], attl, 1e-6), flush=flush), bytes=T * inner * (4 + 2 + 2))
+        y, x, xa = torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda"), prec.empty(T, W)
+        w1 = torch.ones(W, device="cuda")
+        k[f"mapedra_group_norm_residual_{name}"] = dict(s=timed(lambda: seq_ops.group_rmsnorm_add(y, w1, x, xa, 4, 1e-6), flush=flush), bytes=T * W * (4 + 8 + 2))
+        for i in range(n_seq):
+            store.release(("k", i))
+    for name, d in k.items():
+        d["us"] = round(d.pop("s") * 1e6, 2)
+        d["hbm_frac"] = round(d["bytes"] / (d["us"] * 1e-6) / hbm, 4)
+        if "flops" in d:
+            d["tflops"] = round(d["flops"] / (d["us"] * 1e-6) / 1e12, 2)
+            d["tensor_frac"] = round(d["flops"] / (d["us"] * 1e-6) / tflops, 5)
+        bound = max(d["bytes"] / hbm, d.get("flops", 0) / tflops)
+        d["x_roofline"] = round(d["us"] * 1e-6 / bound, 2)
+    out["kernels"] = k
+    out["value"] = out["padulorn_decode_tok_s"]
+    out["unit"] = "tokens/s"
+    out["n_gpus"] = 1
+    for key in list(out):
+        if key.endswith("tok_s"):
+            out[key] = round(out[key], 1)
+    print(json.dumps(out), flush=True)
+    return out

@@ -683,10 +683,11 @@ class RoutedFeedForward:
         return z, ids, wts, plan, self.expert_products(h, plan, counts, prec) if self.n_real else None
 
     def add_normed(self, h, prec, norm_w, x, out_act, eps):
-        """x += N(experts(h)) * norm_w in place (RMS norm), out_act a copy of the new rows: combine, norm and residual in one pass.  For layers
-        without identity outputs and without a shared expert."""
-        if self.shared is not None or self.n_real != self.n_all:
-            raise ValueError("identity outputs and shared experts are not part of the fused combine")
+        """x += N(experts(h)) * norm_w in place (RMS norm), out_act a copy of the new rows.  Combine, norm and residual are one pass for layers
+        without identity outputs and shared expert (and rows that fit the kernel's shared memory)."""
+        if self.shared is not None or self.n_real != self.n_all or self.D > seq_ops.COMBINE_NORM_MAX_WIDTH:
+            seq_ops.group_rmsnorm_add(self(h, None, prec), norm_w, x, out_act, 1, eps)
+            return
         _, _, wts, plan, eo = self._routed(h, prec)
         seq_ops.moe_combine_norm_add(eo, plan, wts, norm_w, x, out_act, eps)
 

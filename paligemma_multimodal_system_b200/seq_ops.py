@@ -597,6 +597,9 @@ def moe_combine(expert_out, plan: MoePlan, ids, weights, h, shared_out, y, share
     return y
 
 
+COMBINE_NORM_MAX_WIDTH = 12288  # a row of sums stays in shared memory
+
+
 def moe_combine_norm_add(expert_out, plan: MoePlan, weights, norm_w, x, out_act, eps):
     """y = sum_k weights[t, k] * expert row; x += y / rms(y) * norm_w in place; out_act (may be None) gets the new row."""
     T, D = x.shape
