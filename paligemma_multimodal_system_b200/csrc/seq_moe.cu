@@ -420,7 +420,8 @@ static int launch_moe_mma(dim3 grid, cudaStream_t st, const void* x, long long l
   return cudaGetLastError() == cudaSuccess ? PG_OK : PG_ERR_CUDA;
 }
 
-// xg[row, :] = x[sorted_pair[row] / top, :] for the `rows` sorted pairs that exist (rows read from offsets[n_real] on the device)
+// xg[row, :] = x[sorted_pair[row] / top, :] for the `rows` sorted pairs that exist (rows read from offsets[n_real] on the device); TA: the
+// piece a thread copies (an element, or 16 bytes of them when rows and pitches allow; D and the pitches count pieces)
 template <typename TA>
 __global__ void moe_gather_rows_kernel(const TA* __restrict__ x, long long ldx, const int* __restrict__ sorted_pair, const int* __restrict__ total,
                                        int top, TA* __restrict__ xg, long long ldg, int D) {
@@ -591,7 +592,10 @@ extern "C" int pg_moe_gather_rows(const void* x, long long ldx, const int* sorte
                                   int max_rows, int D, int act_f32, void* stream) {
   if (max_rows <= 0 || D <= 0 || top <= 0) return PG_ERR_ARG;
   const int grid = max_rows < 16384 ? max_rows : 16384;
-  if (act_f32)
+  const int per = act_f32 ? 4 : 8;  // elements of a 16-byte piece
+  if (D % per == 0 && ldx % per == 0 && ldg % per == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(xg)) & 15) == 0)
+    moe_gather_rows_kernel<uint4><<<grid, 128, 0, PG_ST(stream)>>>(static_cast<const uint4*>(x), ldx / per, sorted_pair, total_rows, top, static_cast<uint4*>(xg), ldg / per, D / per);
+  else if (act_f32)
     moe_gather_rows_kernel<float><<<grid, 128, 0, PG_ST(stream)>>>(static_cast<const float*>(x), ldx, sorted_pair, total_rows, top, static_cast<float*>(xg), ldg, D);
   else
     moe_gather_rows_kernel<bf16><<<grid, 128, 0, PG_ST(stream)>>>(static_cast<const bf16*>(x), ldx, sorted_pair, total_rows, top, static_cast<bf16*>(xg), ldg, D);
