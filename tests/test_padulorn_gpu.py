@@ -293,7 +293,7 @@ def test_head_norm_without_weight_and_silu_gate(rows, groups, size, f32):
     assert bool((buf[:, D:] == 3.0).all())
 
 
-@pytest.mark.parametrize("H,G,dim,vdim,rot", [(4, 2, 24, 20, 12), (6, 3, 64, 64, 64), (3, 1, 9, 5, 4), (2, 2, 96, 64, 24), (1, 1, 2, 1, 2), (8, 2, 128, 128, 0)])
+@pytest.mark.parametrize("H,G,dim,vdim,rot", [(4, 2, 24, 20, 12), (6, 3, 64, 64, 64), (3, 1, 9, 5, 4), (2, 2, 96, 64, 40), (1, 1, 2, 1, 2), (8, 2, 128, 128, 0)])
 @pytest.mark.parametrize("f32", [True, False])
 def test_attention_front_end(H, G, dim, vdim, rot, f32):
     """Norms over the whole projections, rotation with a gain at positions in the thousands, blended values, rows into the right pages."""
@@ -730,7 +730,7 @@ def test_registry_and_command_line_serve_a_checkpoint_folder(tmp_path):
 def test_wider_model_long_prompt_reaches_the_large_tile_paths():
     """Width 512, tensor-core head sizes and per-expert dense products over 1100 tokens in bf16; then 20 decoded tokens beyond the window."""
     cfg = make_cfg([moe(retention(heads=8, dim=64, vdim=64, rot_dims=64), 4, 2, 256, (2, 1)), moe(attention(heads=8, kv_heads=2, dim=64, vdim=64, rot_dims=32, size=300, keep_first=8), 8, 2, 512, (4, 2)),
-                    bare(attention(heads=4, kv_heads=2, dim=96, vdim=64, rot_dims=24, size=None))], width=512, vocab=1000)
+                    bare(attention(heads=6, kv_heads=2, dim=96, vdim=64, rot_dims=48, size=None))], width=512, vocab=1000)
     w = steady_weights(cfg, seed=77)
     tk = toks(1120, 1000, 3)
     ref = O.forward(cfg, w, tk, dtype=F32)
